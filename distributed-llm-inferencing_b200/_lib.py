@@ -15,7 +15,7 @@ LIB_PATH = os.path.join(_HERE, "libdli_b200.so")
 DLI_OK = 0
 EPI_NONE, EPI_BIAS, EPI_RESIDUAL, EPI_GELU_NEW = 0, 1, 2, 4
 
-_vp, _i, _f, _sz = C.c_void_p, C.c_int, C.c_float, C.c_size_t
+_vp, _i, _f, _sz, _ll = C.c_void_p, C.c_int, C.c_float, C.c_size_t, C.c_longlong
 
 # name -> (restype, argtypes); mirrors include/dli.h one to one
 SIGNATURES = {
@@ -70,7 +70,7 @@ SIGNATURES = {
     "dli_gemv_argmax_bf16": (_i, [_vp, _vp, _f, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _vp, _sz, _vp]),
     "dli_sample_bf16": (_i, [_vp, _i, _vp, _i, _i, _f, _i, _f, _vp, _vp, _vp, _vp, _i, _vp]),
     "dli_decode_advance": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _vp]),
-    "dli_embedding_f32": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp, _vp, _vp, _vp]),
+    "dli_embedding_f32": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp, _vp, _vp, _vp, _i, _ll, _ll, _vp, _i, _sz, _vp]),
     "dli_group_rmsnorm": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp]),
     "dli_group_rmsnorm_conv_single": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _vp]),
     "dli_residual_add2": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp]),
@@ -86,7 +86,7 @@ SIGNATURES = {
     "dli_ssm_scan_ragged": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _vp, _i, _vp]),
     "dli_ssm_parallel_scratch_floats": (_sz, [_i, _i, _i, _i]),
     "dli_gated_group_rmsnorm": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _i, _vp]),
-    "dli_moe_route": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp]),
+    "dli_moe_route": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp]),
     "dli_moe_sel_supported": (_i, [_i, _i, _i, _i]),
     "dli_moe_sel_bf16": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _f, _f, _i, _vp]),
     "dli_moe_act": (_i, [_vp, _vp, _vp, _i, _i, _i, _f, _i, _f, _f, _i, _i, _i, _vp]),
@@ -96,23 +96,28 @@ SIGNATURES = {
     "dli_postnorm_add_norm_conv_single": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _f, _f, _i, _vp]),
     "dli_gather_cast": (_i, [_vp, _vp, _vp, _i, _i, _i, _vp]),
     "dli_linear_any": (_i, [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp]),
-    "dli_silu_mul": (_i, [_vp, _vp, _i, _i, _i, _i, _vp, _vp]),
+    "dli_silu_mul": (_i, [_vp, _vp, _i, _i, _i, _i, _vp, _i, _vp]),
     "dli_attn_prep_append": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i,
-                                  _vp, _vp, _f, _vp, _vp, _vp, _vp, _i, _i, _vp, _i, _vp]),
+                                  _vp, _vp, _f, _vp, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _vp]),
     "dli_attn_ragged": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _vp, _i,
-                             _i, _vp, _vp, _i, _i, _vp, _i, _vp, _vp, _vp]),
+                             _i, _vp, _vp, _i, _i, _vp, _i, _vp, _vp, _f, _i, _f, _i, _vp]),
     "dli_attn_ragged_tc_supported": (_i, [_i, _i, _i]),
     "dli_attn_ragged_tc": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _vp, _i,
-                                _i, _vp, _vp, _vp, _vp, _vp]),
+                                _i, _vp, _vp, _vp, _vp, _f, _i, _f, _i, _vp]),
     "dli_layer_close": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _sz, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i,
-                             _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _vp]),
+                             _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _vp, _vp]),
     "dli_token_shift_ragged": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp]),
     "dli_postnorm_vec_add": (_i, [_vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp]),
     "dli_token_side_act": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp]),
     "dli_token_side_gate": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
     "dli_token_side": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp]),
     "dli_delta_rule_ragged": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _f, _i, _i, _vp]),
-    "dli_head_rmsnorm_gate": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _i, _i, _i, _vp]),
+    "dli_head_rmsnorm_gate": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _i, _i, _i, _i, _vp]),
+    "dli_streams_close": (_i, [_vp, _vp, _sz, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp, _vp, _vp, _vp, _vp, _vp,
+                               _vp, _i, _i, _i, _i, _i, _f, _i, _vp]),
+    "dli_linattn_scratch_floats": (_sz, [_i, _i, _i, _i]),
+    "dli_linattn_ragged": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _vp, _i, _vp, _i, _i,
+                                _vp, _vp, _f, _i, _vp, _vp, _i, _vp, _i, _vp]),
     "dli_mlstm_parallel_scratch_floats": (_sz, [_i, _i, _i, _i]),
     "dli_mlstm_ragged_parallel": (_i, [_vp, _vp, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i,
                                        _vp, _vp, _f, _vp, _f, _vp, _vp, _vp, _i, _vp]),

@@ -37,6 +37,8 @@ SOURCES = [
     "moe.cu",
     "delta_rule.cu",
     "prenorm_rows.cu",
+    "stream_rows.cu",
+    "linear_attn.cu",
 ]
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]

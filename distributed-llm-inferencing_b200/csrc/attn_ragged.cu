@@ -12,7 +12,10 @@
 //   - an output gate: head h's output times sigmoid(gate[row, h]),
 //   - biases on the q / k / v projections (added here, in fp32, before norm and rotation), a layer that only makes
 //     queries and reads ANOTHER layer's cached keys and values,
-//   - a distance penalty: r1[h] * ln(1 + r2[h] * (i - j)) is taken off the scaled score of query i and key j.
+//   - a distance penalty: r1[h] * ln(1 + r2[h] * (i - j)) is taken off the scaled score of query i and key j,
+//   - a soft cap on the scaled scores, cap * tanh(score / cap); rotation of pairs (i, i + rd/2) instead of (2i, 2i+1);
+//     an output gate per CHANNEL, sigmoid(gate[row, h*V + v]); a factor on the output; output rows that are part of
+//     wider rows (mixers that share one output projection).
 // Scores, softmax weights and the accumulation are fp32; the cache holds E (bf16 or float).
 //
 // Step description as in ragged_rows.cu: row_ent[rows], ent[4 * n_ent] = (slot, first row, rows, first position);
@@ -47,6 +50,7 @@ struct AttnPrep {
   int table_len;
   const float* bias;        // [>= the projection's q / k / v columns] fp32 or NULL: added to the projection's columns
   int q_only;               // 1: only the queries are made; keys and values are another layer's
+  int halves;               // rotation pairs: 0: (2i, 2i+1), 1: (i, i + rd/2)
 };
 
 // One CTA per row; each warp takes heads in turn: q heads -> qbuf (fp32, normed and rotated), key heads and value
@@ -82,16 +86,19 @@ attn_prep_append_kernel(const E* __restrict__ proj, float* __restrict__ qbuf, E*
       float* qd = qbuf + ((size_t)row * a.H + hh) * a.D;
       E* kd = kc + (((size_t)page * a.G + hh) * a.page_size + off) * a.D;
       for (int i = lane; i < a.D / 2; i += 32) {
-        float u = a_to_f(src[2 * i]), v = a_to_f(src[2 * i + 1]);
-        if (bs) { u += bs[2 * i]; v += bs[2 * i + 1]; }
-        if (nw) { u = u * r * nw[2 * i]; v = v * r * nw[2 * i + 1]; }
+        // the pair's two dimensions; pairs behind the rotated ones are neighbours in both layouts
+        const bool half_pair = a.halves && 2 * i < a.rd;
+        const int i0 = half_pair ? i : 2 * i, i1 = half_pair ? i + a.rd / 2 : 2 * i + 1;
+        float u = a_to_f(src[i0]), v = a_to_f(src[i1]);
+        if (bs) { u += bs[i0]; v += bs[i1]; }
+        if (nw) { u = u * r * nw[i0]; v = v * r * nw[i1]; }
         if (a.cos_qk && 2 * i < a.rd) {
           const float c = a.cos_qk[(size_t)pos * (a.rd / 2) + i], s = a.sin_qk[(size_t)pos * (a.rd / 2) + i];
           const float u2 = u * c - v * s, v2 = v * c + u * s;
           u = u2; v = v2;
         }
-        if (is_q) { qd[2 * i] = u; qd[2 * i + 1] = v; }
-        else { kd[2 * i] = a_from_f<E>(u); kd[2 * i + 1] = a_from_f<E>(v); }
+        if (is_q) { qd[i0] = u; qd[i1] = v; }
+        else { kd[i0] = a_from_f<E>(u); kd[i1] = a_from_f<E>(v); }
       }
     } else {
       const int g = item - a.H - a.G;
@@ -131,7 +138,19 @@ struct AttnRun {
   float* part;              // [rows, H, splits, V + 2] (unnormalised output, maximum, denominator) a merge kernel adds
   const float* r1;          // [H] or NULL: the distance penalty r1[h] * ln(1 + r2[h] * (i - j)) on the scaled scores
   const float* r2;
+  float cap;                // > 0: scores become cap * tanh(score / cap) (before the penalty's place in the order: not combined)
+  int g_chan;               // 1: the gate's columns are one per output channel, g_off + h*V + v
+  float oscale;             // factor on the output
+  int ldo;                  // elements between output rows
 };
+
+// sigmoid gate of output channel d of head h (1 without a gate); the per-head gate is the same for every d
+template <typename E>
+__device__ __forceinline__ float out_gate(const E* proj, const AttnRun& a, size_t row, int h, int d) {
+  if (a.g_off < 0) return a.oscale;
+  const float z = a_to_f(proj[row * a.ldp + a.g_off + (a.g_chan ? h * a.V + d : h)]);
+  return a.oscale / (1.f + expf(-z));
+}
 
 // q (shared, fp32) . k row (global): 16-byte loads where the row allows them
 __device__ __forceinline__ float dot_row(const float* q, const bf16* kr, int D) {
@@ -246,6 +265,7 @@ attn_ragged_kernel(const float* __restrict__ qbuf, const E* __restrict__ kc, con
       }
       if (tpk > 1) dpart += __shfl_xor_sync(0xffffffffu, dpart, 1);
       if (tpk > 2) dpart += __shfl_xor_sync(0xffffffffu, dpart, 2);
+      if (a.cap > 0.f) dpart = a.cap * tanhf(dpart / a.cap);
       if (j <= je && part == 0) s = a.r1 ? dpart - pen1 * log1pf(pen2 * (float)(pos - jp)) : dpart;
     }
     // block maximum
@@ -322,10 +342,8 @@ attn_ragged_kernel(const float* __restrict__ qbuf, const E* __restrict__ kc, con
     if (tid == 0) { pr[a.V] = m; pr[a.V + 1] = l; }
     return;
   }
-  float gate = 1.f;
-  if (a.g_off >= 0) gate = 1.f / (1.f + expf(-a_to_f(proj[(size_t)row * a.ldp + a.g_off + h])));
   const float inv = 1.f / l;
-  E* orow = out + ((size_t)row * a.H + h) * a.V;
+  E* orow = out + (size_t)row * a.ldo + h * a.V;
   for (int i = tid; i < a.V / 2; i += kAttnThreads) {
     float u = 0.f, v = 0.f;
     for (int gg = 0; gg < groups; ++gg) { u += ov[gg * a.V + 2 * i]; v += ov[gg * a.V + 2 * i + 1]; }
@@ -335,8 +353,8 @@ attn_ragged_kernel(const float* __restrict__ qbuf, const E* __restrict__ kc, con
       const float u2 = u * c + v * s, v2 = v * c - u * s;  // by -angle
       u = u2; v = v2;
     }
-    orow[2 * i] = a_from_f<E>(u * gate);
-    orow[2 * i + 1] = a_from_f<E>(v * gate);
+    orow[2 * i] = a_from_f<E>(u * out_gate(proj, a, row, h, 2 * i));
+    orow[2 * i + 1] = a_from_f<E>(v * out_gate(proj, a, row, h, 2 * i + 1));
   }
 }
 
@@ -365,10 +383,8 @@ attn_ragged_merge_kernel(const E* __restrict__ proj, E* __restrict__ out, AttnRu
   for (int z = 0; z < a.splits; ++z) L += wz[z] * lz[z];
   const int4 e = reinterpret_cast<const int4*>(a.ent)[a.row_ent[row]];
   const int pos = e.w + (row - e.y);
-  float gate = 1.f;
-  if (a.g_off >= 0) gate = 1.f / (1.f + expf(-a_to_f(proj[(size_t)row * a.ldp + a.g_off + h])));
   const float inv = 1.f / L;
-  E* orow = out + ((size_t)row * a.H + h) * a.V;
+  E* orow = out + (size_t)row * a.ldo + h * a.V;
   for (int i = tid; i < a.V / 2; i += kAttnThreads) {
     float u = 0.f, v = 0.f;
     for (int z0 = 0; z0 < a.splits; z0 += 8) {  // eight splits' loads in flight together
@@ -388,8 +404,8 @@ attn_ragged_merge_kernel(const E* __restrict__ proj, E* __restrict__ out, AttnRu
       const float u2 = u * c + v * s, v2 = v * c - u * s;
       u = u2; v = v2;
     }
-    orow[2 * i] = a_from_f<E>(u * gate);
-    orow[2 * i + 1] = a_from_f<E>(v * gate);
+    orow[2 * i] = a_from_f<E>(u * out_gate(proj, a, row, h, 2 * i));
+    orow[2 * i + 1] = a_from_f<E>(v * out_gate(proj, a, row, h, 2 * i + 1));
   }
 }
 
@@ -563,8 +579,8 @@ static int launch_shared_kv(const float* qbuf, const void* kc, const void* vc, v
 
 // Does a step of this shape take the shared-key/value kernel, and with how many heads per CTA (0: no)?
 static int shared_kv_heads(int H, int G, int D, int V, int ldv, int chunk, int window, int g_off, const float* cos_v, int dt,
-                           const void* kc, const void* vc, bool has_penalty) {
-  if (G != 1 || H < 2 || chunk > 0 || window > 0 || g_off >= 0 || cos_v || has_penalty) return 0;
+                           const void* kc, const void* vc, bool plain_only) {
+  if (G != 1 || H < 2 || chunk > 0 || window > 0 || g_off >= 0 || cos_v || plain_only) return 0;
   const size_t es = dt == 0 ? 2 : 4;
   if (D % 8 != 0 || !attn_vec_values(V, ldv) || (ldv * es) % (dt == 0 ? 8 : 16) != 0 || !aligned16(kc) ||
       (reinterpret_cast<uintptr_t>(vc) & 15u) != 0)
@@ -663,6 +679,8 @@ attn_ragged_tc_kernel(const float* __restrict__ qbuf, const bf16* __restrict__ k
   // the distance penalty in the softmax's base-2 exponent: r1 ln(1 + r2 d) log2(e) = r1 log2(1 + r2 d); the scores stay
   // raw dot products, so it is taken off as pen / scale_log2
   const float pen1 = a.r1 ? a.r1[h] / scale_log2 : 0.f, pen2 = a.r1 ? a.r2[h] : 0.f;
+  // the soft cap on raw dot products: (cap / scale) * tanh(s * scale / cap), the hyperbolic tangent as 1 - 2 / (e^(2x) + 1)
+  const float cap_raw = a.cap > 0.f ? a.cap / a.scale : 0.f, cap_in = a.cap > 0.f ? 2.f * scale_log2 / a.cap : 0.f;
   float m_run[2] = {m0, m0};
   float l_run[2] = {(a.sink && t4 == 0) ? 1.f : 0.f, (a.sink && t4 == 0) ? 1.f : 0.f};
   float o[DV / 8][4];
@@ -705,6 +723,13 @@ attn_ragged_tc_kernel(const float* __restrict__ qbuf, const bf16* __restrict__ k
       }
     }
     const int tk0 = tile * kRtTile;
+    if (a.cap > 0.f) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+          s[j][x] = cap_raw * (1.f - __fdividef(2.f, ex2_ftz(fminf(s[j][x] * cap_in, 100.f)) + 1.f));
+    }
     if (a.r1) {
 #pragma unroll
       for (int j = 0; j < 8; ++j)
@@ -773,8 +798,9 @@ attn_ragged_tc_kernel(const float* __restrict__ qbuf, const bf16* __restrict__ k
       const size_t row = (size_t)e.y + q0 + lr;
       const int pos = qabs[r];
       float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;
-      if (a.g_off >= 0) inv *= 1.f / (1.f + expf(-__bfloat162float(proj[row * a.ldp + a.g_off + h])));
-      bf16* dst = out + (row * a.H + h) * DV + 2 * t4;
+      inv *= a.g_chan ? a.oscale : out_gate(proj, a, row, h, 0);
+      bf16* dst = out + row * a.ldo + h * DV + 2 * t4;
+      const bf16* gsrc = a.g_chan ? proj + row * a.ldp + a.g_off + h * DV + 2 * t4 : nullptr;
 #pragma unroll
       for (int i = 0; i < DV / 8; ++i) {
         float u = o[i][2 * r], v = o[i][2 * r + 1];
@@ -783,6 +809,10 @@ attn_ragged_tc_kernel(const float* __restrict__ qbuf, const bf16* __restrict__ k
           const float c = a.cos_v[(size_t)pos * (DV / 2) + pr], sn = a.sin_v[(size_t)pos * (DV / 2) + pr];
           const float u2 = u * c + v * sn, v2 = v * c - u * sn;
           u = u2; v = v2;
+        }
+        if (a.g_chan) {
+          u = __fdividef(u, 1.f + ex2_ftz(-1.4426950408889634f * __bfloat162float(gsrc[i * 8])));
+          v = __fdividef(v, 1.f + ex2_ftz(-1.4426950408889634f * __bfloat162float(gsrc[i * 8 + 1])));
         }
         *reinterpret_cast<uint32_t*>(dst + i * 8) = pack_bf16(u * inv, v * inv);
       }
@@ -812,7 +842,8 @@ int dli_attn_prep_append(const void* proj, float* qbuf, void* k_cache, void* v_c
                          const int32_t* ent, const int32_t* page_table, int max_pages, int page_size, int rows, int H,
                          int G, int D, int V, int rd, int ldp, int q_off, int k_off, int v_off, const float* q_norm,
                          const float* k_norm, float eps, const float* cos_qk, const float* sin_qk, const float* cos_v,
-                         const float* sin_v, int table_len, int dt, const float* bias, int q_only, dli_stream_t stream) {
+                         const float* sin_v, int table_len, int dt, const float* bias, int q_only, int halves,
+                         dli_stream_t stream) {
   DLI_CHECK_ARG(proj && qbuf && (q_only || (k_cache && v_cache)) && row_ent && ent && page_table, "dli_attn_prep_append: null pointer");
   DLI_CHECK_ARG(H > 0 && G > 0 && H % G == 0 && D > 0 && V > 0 && D % 2 == 0 && V % 2 == 0 && rd % 2 == 0 && rd <= D,
                 "dli_attn_prep_append: H=%d G=%d D=%d V=%d rd=%d (H %% G == 0, even sizes, rd <= D)", H, G, D, V, rd);
@@ -820,7 +851,7 @@ int dli_attn_prep_append(const void* proj, float* qbuf, void* k_cache, void* v_c
   DLI_CHECK_ARG(dt == 0 || dt == 1, "element type %d: 0 = bf16, 1 = float", dt);
   if (rows <= 0) return DLI_OK;
   AttnPrep a{row_ent, ent, page_table, max_pages, page_size, H, G, D, V, rd, ldp, q_off, k_off, v_off, q_norm, k_norm,
-             eps, (rd > 0 ? cos_qk : nullptr), sin_qk, cos_v, sin_v, table_len, bias, q_only ? 1 : 0};
+             eps, (rd > 0 ? cos_qk : nullptr), sin_qk, cos_v, sin_v, table_len, bias, q_only ? 1 : 0, halves ? 1 : 0};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int items = q_only ? H : H + 2 * G;
   const dim3 pgrid(rows, rows <= 64 ? (items + 3) / 4 : 1);
@@ -833,7 +864,7 @@ int dli_attn_ragged(const float* qbuf, const void* k_cache, const void* v_cache,
                     const int32_t* row_ent, const int32_t* ent, const int32_t* page_table, int max_pages, int page_size,
                     int rows, int H, int G, int D, int V, float scale, int chunk, int window, int first, const float* sink,
                     int ldp, int g_off, const float* cos_v, const float* sin_v, int ldv, int splits, float* part, int dt,
-                    const float* r1, const float* r2, dli_stream_t stream) {
+                    const float* r1, const float* r2, float cap, int g_chan, float out_scale, int ldo, dli_stream_t stream) {
   DLI_CHECK_ARG(qbuf && k_cache && v_cache && out && row_ent && ent && page_table, "dli_attn_ragged: null pointer");
   DLI_CHECK_ARG(splits >= 1 && splits <= 64 && (splits == 1 || part), "dli_attn_ragged: %d key splits (1..64, with scratch)", splits);
   DLI_CHECK_ARG(ldv == 0 || ldv >= V, "dli_attn_ragged: value row stride %d is below the value size %d", ldv, V);
@@ -845,13 +876,16 @@ int dli_attn_ragged(const float* qbuf, const void* k_cache, const void* v_cache,
   if (rows <= 0) return DLI_OK;
   DLI_CHECK_ARG(first >= 0, "dli_attn_ragged: %d kept first positions", first);
   DLI_CHECK_ARG((r1 == nullptr) == (r2 == nullptr), "dli_attn_ragged: the distance penalty needs both r1 and r2");
+  DLI_CHECK_ARG(ldo == 0 || ldo >= H * V, "dli_attn_ragged: output row stride %d is below %d", ldo, H * V);
+  g_chan = g_off >= 0 && g_chan;
   AttnRun a{row_ent, ent, page_table, max_pages, page_size, H, G, D, V, scale, chunk, window, first, sink, ldp, g_off, cos_v,
-            sin_v, ldv ? ldv : V, splits, part, r1, r2};
+            sin_v, ldv ? ldv : V, splits, part, r1, r2, cap > 0.f ? cap : 0.f, g_chan, out_scale, ldo ? ldo : H * V};
   const int groups = attn_value_groups(V, ldv ? ldv : V);
   const size_t smem = sizeof(float) * (D + kAttnThreads + 8 + (size_t)groups * V);
   DLI_CHECK_ARG(smem <= 48 * 1024, "dli_attn_ragged: key size %d needs %zu bytes of shared memory", D, smem);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const int hpc = shared_kv_heads(H, G, D, V, ldv ? ldv : V, chunk, window, g_off, cos_v, dt, k_cache, v_cache, r1 != nullptr);
+  const int hpc = shared_kv_heads(H, G, D, V, ldv ? ldv : V, chunk, window, g_off, cos_v, dt, k_cache, v_cache,
+                                  r1 != nullptr || cap > 0.f || out_scale != 1.f || a.ldo != H * V);
   if (hpc) {
     int rc;
     if (dt == 0) rc = hpc == 4 ? launch_shared_kv<bf16, 4>(qbuf, k_cache, v_cache, out, rows, a, s)
@@ -878,7 +912,7 @@ int dli_attn_ragged_tc(const float* qbuf, const void* k_cache, const void* v_cac
                        const int32_t* ent, const int32_t* tiles, int n_tiles, const int32_t* page_table, int max_pages,
                        int page_size, int H, int G, int D, int V, float scale, int chunk, int window, int first,
                        const float* sink, int ldp, int g_off, const float* cos_v, const float* sin_v, const float* r1,
-                       const float* r2, dli_stream_t stream) {
+                       const float* r2, float cap, int g_chan, float out_scale, int ldo, dli_stream_t stream) {
   DLI_CHECK_ARG(qbuf && k_cache && v_cache && out && ent && tiles && page_table, "dli_attn_ragged_tc: null pointer");
   DLI_CHECK_ARG(g_off < 0 || proj, "dli_attn_ragged_tc: a gate needs the projection rows");
   DLI_CHECK_ARG(H > 0 && G > 0 && H % G == 0 && scale > 0.f, "dli_attn_ragged_tc: H=%d G=%d scale=%g", H, G, scale);
@@ -887,7 +921,9 @@ int dli_attn_ragged_tc(const float* qbuf, const void* k_cache, const void* v_cac
   if (n_tiles <= 0) return DLI_OK;
   DLI_CHECK_ARG(first >= 0, "dli_attn_ragged_tc: %d kept first positions", first);
   DLI_CHECK_ARG((r1 == nullptr) == (r2 == nullptr), "dli_attn_ragged_tc: the distance penalty needs both r1 and r2");
-  AttnRun a{nullptr, ent, page_table, max_pages, page_size, H, G, D, V, scale, chunk, window, first, sink, ldp, g_off, cos_v, sin_v, V, 1, nullptr, r1, r2};
+  DLI_CHECK_ARG(ldo == 0 || (ldo >= H * V && ldo % 2 == 0), "dli_attn_ragged_tc: output row stride %d (even, at least %d)", ldo, H * V);
+  AttnRun a{nullptr, ent, page_table, max_pages, page_size, H, G, D, V, scale, chunk, window, first, sink, ldp, g_off, cos_v, sin_v, V, 1, nullptr, r1, r2,
+            cap > 0.f ? cap : 0.f, g_off >= 0 && g_chan ? 1 : 0, out_scale, ldo ? ldo : H * V};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (D == 64 && V == 64) return launch_ragged_tc<64, 64>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);
   if (D == 128 && V == 128) return launch_ragged_tc<128, 128>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);

@@ -11,7 +11,7 @@
 // S^T [slots, H, V, D], so that a warp reads and writes its columns as contiguous runs.
 //   dli_delta_rule_ragged   qkv fp32 [rows, 2*G*D + H*V] (q | k | v after their convolutions and activations),
 //                           b_t / a_t columns of the projection row -> o fp32 [rows, H*V]; state read and advanced
-//   dli_head_rmsnorm_gate   out[row, h, :] = o / sqrt(mean(o^2) + eps) * w * act(gate[row, h, :])
+//   dli_head_rmsnorm_gate   out[row, h, :] = o / sqrt(mean(o^2) + eps) * w * act(gate[row, h, :]), w optional
 // Everything is fp32 except the projection row (b, a, gate) and the output, which have the engine's element type.
 // An entry whose first position is 0 starts from a zero state whatever its slot held before.
 #include <math.h>
@@ -446,32 +446,97 @@ delta_rule_block_kernel(const float* __restrict__ qkv, const E* __restrict__ pro
   }
 }
 
-// One warp per (row, head): RMS norm over the head's V outputs, weight, gate.  w_heads != 0: w is [H, V], else [V]
-// shared by the heads.  gate: 0 none, 1 SiLU, 2 sigmoid of proj[row, g_off + h*V + v].
-template <typename E>
-__global__ void __launch_bounds__(256)
+// RMS norm over the head's V outputs, weight, gate.  w: NULL (no weight), [V] shared by the heads, or [H, V] (w_heads != 0).
+// gate: 0 none, 1 SiLU, 2 sigmoid of proj[row, g_off + h*V + v].  ldo: elements between output rows.  `group` threads share a
+// (row, head): a warp each (8 per CTA) for head-sized V, the whole CTA where V is a row (heads normed together).  VEC
+// consecutive channels per thread and access.
+struct HeadNorm {
+  int rows, H, V;
+  float eps;
+  int w_heads, gate, ldp, g_off, ldo;
+};
+
+template <typename E, int VEC, bool kWide>
+__global__ void __launch_bounds__(1024)
 head_rmsnorm_gate_kernel(const float* __restrict__ o, const E* __restrict__ proj, const float* __restrict__ w,
-                         E* __restrict__ out, int rows, int H, int V, float eps, int w_heads, int gate, int ldp,
-                         int g_off) {
+                         E* __restrict__ out, HeadNorm a) {
+  __shared__ float red[32];
   pdl_wait();
   pdl_trigger();
   const int lane = threadIdx.x & 31;
-  const size_t item = (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (item >= (size_t)rows * H) return;
-  const size_t row = item / H;
-  const int h = (int)(item - row * H);
-  const float* src = o + item * V;
+  const int me = kWide ? threadIdx.x : lane, group = kWide ? blockDim.x : 32;
+  const size_t item = kWide ? (size_t)blockIdx.x : (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (item >= (size_t)a.rows * a.H) return;
+  const size_t row = item / a.H;
+  const int h = (int)(item - row * a.H);
+  const float* src = o + item * a.V;
   float ss = 0.f;
-  for (int v = lane; v < V; v += 32) ss = fmaf(src[v], src[v], ss);
-  const float r = 1.f / sqrtf(warp_sum(ss) / V + eps);
-  for (int v = lane; v < V; v += 32) {
-    float y = src[v] * r * w[w_heads ? h * V + v : v];
-    if (gate) {
-      const float z = d_to_f(proj[row * ldp + g_off + h * V + v]);
-      y *= gate == 1 ? z / (1.f + expf(-z)) : 1.f / (1.f + expf(-z));
+  for (int v = me * VEC; v < a.V; v += group * VEC) {
+    if constexpr (VEC == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(src + v);
+      ss = fmaf(f.x, f.x, ss); ss = fmaf(f.y, f.y, ss); ss = fmaf(f.z, f.z, ss); ss = fmaf(f.w, f.w, ss);
+    } else {
+      ss = fmaf(src[v], src[v], ss);
     }
-    out[item * V + v] = d_from_f<E>(y);
   }
+  ss = warp_sum(ss);
+  if (kWide) {
+    if (lane == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+    for (int i = 0; i < (int)(blockDim.x >> 5); ++i) ss += red[i];
+  }
+  const float r = 1.f / sqrtf(ss / a.V + a.eps);
+  const E* gp = a.gate ? proj + row * a.ldp + a.g_off + h * a.V : nullptr;
+  const float* wp = w ? w + (a.w_heads ? h * a.V : 0) : nullptr;
+  E* dst = out + row * a.ldo + h * a.V;
+  auto gated = [&](float y, float z) {
+    return a.gate == 1 ? y * (z / (1.f + expf(-z))) : y / (1.f + expf(-z));
+  };
+  for (int v = me * VEC; v < a.V; v += group * VEC) {
+    if constexpr (VEC == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(src + v);
+      float y[4] = {f.x * r, f.y * r, f.z * r, f.w * r};
+      if (wp) {
+        const float4 w4 = *reinterpret_cast<const float4*>(wp + v);
+        y[0] *= w4.x; y[1] *= w4.y; y[2] *= w4.z; y[3] *= w4.w;
+      }
+      if (a.gate) {
+        float z[4];
+        if constexpr (sizeof(E) == 2) {
+          const uint2 u = *reinterpret_cast<const uint2*>(gp + v);
+          z[0] = bf_lo(u.x); z[1] = bf_hi(u.x); z[2] = bf_lo(u.y); z[3] = bf_hi(u.y);
+        } else {
+          const float4 z4 = *reinterpret_cast<const float4*>(gp + v);
+          z[0] = z4.x; z[1] = z4.y; z[2] = z4.z; z[3] = z4.w;
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) y[i] = gated(y[i], z[i]);
+      }
+      if constexpr (sizeof(E) == 2) *reinterpret_cast<uint2*>(dst + v) = make_uint2(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]));
+      else *reinterpret_cast<float4*>(dst + v) = make_float4(y[0], y[1], y[2], y[3]);
+    } else {
+      float y = src[v] * r;
+      if (wp) y *= wp[v];
+      if (a.gate) y = gated(y, d_to_f(gp[v]));
+      dst[v] = d_from_f<E>(y);
+    }
+  }
+}
+
+template <typename E>
+static int launch_head_norm(const float* o, const void* proj, const float* w, void* out, const HeadNorm& a, cudaStream_t s) {
+  const uintptr_t ea = 4 * sizeof(E) - 1;  // four elements as one access
+  const bool vec = a.V % 4 == 0 && a.ldo % 4 == 0 && aligned16(o) && (!w || aligned16(w)) && (reinterpret_cast<uintptr_t>(out) & ea) == 0 &&
+                   (!a.gate || (a.ldp % 4 == 0 && a.g_off % 4 == 0 && (reinterpret_cast<uintptr_t>(proj) & ea) == 0));
+  const bool wide = a.V >= 1024;
+  const unsigned items = (unsigned)((size_t)a.rows * a.H);
+  const dim3 grid(wide ? items : (items + 7) / 8), block(wide && items <= 64 && a.V >= 4096 ? 1024 : 256);
+#define HN_LAUNCH(VEC, W) DLI_LAUNCH("head_rmsnorm_gate", (head_rmsnorm_gate_kernel<E, VEC, W>), grid, block, 0, s, o, (const E*)proj, w, (E*)out, a)
+  if (vec) { if (wide) HN_LAUNCH(4, true); else HN_LAUNCH(4, false); }
+  else { if (wide) HN_LAUNCH(1, true); else HN_LAUNCH(1, false); }
+#undef HN_LAUNCH
+  return DLI_OK;
 }
 
 template <typename E, int CPT, int NS>
@@ -535,16 +600,14 @@ int dli_delta_rule_ragged(const float* qkv, const void* proj, float* St, float* 
 }
 
 int dli_head_rmsnorm_gate(const float* o, const void* proj, const float* w, void* out, int rows, int H, int V, float eps,
-                          int w_heads, int gate, int ldp, int g_off, int dt, dli_stream_t stream) {
-  DLI_CHECK_ARG(o && w && out && (gate == 0 || proj) && gate >= 0 && gate <= 2 && H > 0 && V > 0,
+                          int w_heads, int gate, int ldp, int g_off, int ldo, int dt, dli_stream_t stream) {
+  DLI_CHECK_ARG(o && out && (gate == 0 || proj) && gate >= 0 && gate <= 2 && H > 0 && V > 0 && (ldo == 0 || ldo >= H * V),
                 "dli_head_rmsnorm_gate: null pointer or bad shape");
   DLI_CHECK_ARG(dt == 0 || dt == 1, "element type %d: 0 = bf16, 1 = float", dt);
   if (rows <= 0) return DLI_OK;
+  HeadNorm a{rows, H, V, eps, w_heads, gate, ldp, g_off, ldo ? ldo : H * V};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const unsigned grid = (unsigned)(((size_t)rows * H + 7) / 8);
-  if (dt == 0) DLI_LAUNCH("head_rmsnorm_gate", head_rmsnorm_gate_kernel<bf16>, dim3(grid), dim3(256), 0, s, o, (const bf16*)proj, w, (bf16*)out, rows, H, V, eps, w_heads, gate, ldp, g_off);
-  else DLI_LAUNCH("head_rmsnorm_gate", head_rmsnorm_gate_kernel<float>, dim3(grid), dim3(256), 0, s, o, (const float*)proj, w, (float*)out, rows, H, V, eps, w_heads, gate, ldp, g_off);
-  return DLI_OK;
+  return dt == 0 ? launch_head_norm<bf16>(o, proj, w, out, a, s) : launch_head_norm<float>(o, proj, w, out, a, s);
 }
 
 }  // extern "C"

@@ -13,6 +13,7 @@
 //                   expert's routing weight, so that ONE down projection over the concatenated experts is the
 //                   weighted sum of their outputs.  A shared expert (its own size and limit, weight 1) is the last
 //                   block.  mode 1: experts without a gate, a = max(u, 0)^2 on the stacked up projections.
+//                   mode 2: a = silu(g) * u, no limits.
 #include <math.h>
 
 #include "common.cuh"
@@ -43,9 +44,17 @@ struct MoeAct {
   float limit_s;
   float alpha;              // g * sigmoid(alpha * g)
   int ld;                   // row stride of gu
-  int mode;                 // 0: clamped gated form; 1: no gate, max(u, 0)^2, columns [e*ff, +ff) of gu (shared: after them)
-  int vec;                  // mode 1: sizes and pointers allow 16-byte accesses
+  int mode;                 // 0: clamped gated form; 1: no gate, max(u, 0)^2, columns [e*ff, +ff) of gu (shared: after them); 2: silu(g) * u
+  int vec;                  // modes 1 and 2: sizes and pointers allow 16-byte accesses
 };
+
+// one gated activation, modes 0 and 2
+__device__ __forceinline__ float moe_gated(float g, float u, float lim, const MoeAct& a) {
+  if (a.mode == 2) return g / (1.f + expf(-g)) * u;
+  g = fminf(g, lim);
+  u = fminf(fmaxf(u, -lim), lim);
+  return g / (1.f + expf(-a.alpha * g)) * (u + 1.f);
+}
 
 // act[row, e*ff + f] and act[row, n_exp*ff + f] (shared); a row's channels go to one CTA, or to several for few rows.
 template <typename E>
@@ -83,6 +92,35 @@ moe_act_kernel(const E* __restrict__ gu, const float* __restrict__ wts, E* __res
     }
     return;
   }
+  if (a.mode == 2 && a.vec) {
+    // gated experts, 16 bytes per thread and access of the gate and of the up columns
+    constexpr int V = 16 / (int)sizeof(E);
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * V; i < F; i += blockDim.x * gridDim.y * V) {
+      const bool routed = i < a.n_exp * a.ff;
+      const int e = routed ? i / a.ff : a.n_exp, f = i - e * a.ff, ff = routed ? a.ff : a.ff_s;
+      const float wt = routed ? wts[row * a.n_exp + e] : 1.f;
+      uint4 o = make_uint4(0, 0, 0, 0);
+      if (wt != 0.f) {
+        const E* gp = g + (size_t)e * 2 * a.ff + f;
+        const uint4 gu4 = *reinterpret_cast<const uint4*>(gp), uu4 = *reinterpret_cast<const uint4*>(gp + ff);
+        if constexpr (sizeof(E) == 2) {
+          float gf[8], uf[8];
+          unpack8(gu4, gf);
+          unpack8(uu4, uf);
+#pragma unroll
+          for (int k = 0; k < 8; ++k) gf[k] = moe_gated(gf[k], uf[k], 0.f, a) * wt;
+          o = pack8(gf);
+        } else {
+          o.x = __float_as_uint(moe_gated(__uint_as_float(gu4.x), __uint_as_float(uu4.x), 0.f, a) * wt);
+          o.y = __float_as_uint(moe_gated(__uint_as_float(gu4.y), __uint_as_float(uu4.y), 0.f, a) * wt);
+          o.z = __float_as_uint(moe_gated(__uint_as_float(gu4.z), __uint_as_float(uu4.z), 0.f, a) * wt);
+          o.w = __float_as_uint(moe_gated(__uint_as_float(gu4.w), __uint_as_float(uu4.w), 0.f, a) * wt);
+        }
+      }
+      *reinterpret_cast<uint4*>(out + i) = o;
+    }
+    return;
+  }
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < F; i += blockDim.x * gridDim.y) {
     float gv, uv, lim, wt;
     if (a.mode == 1) {
@@ -109,10 +147,7 @@ moe_act_kernel(const E* __restrict__ gu, const float* __restrict__ wts, E* __res
       uv = x_to_f(g[(size_t)a.n_exp * 2 * a.ff + a.ff_s + f]);
       lim = a.limit_s;
     }
-    gv = fminf(gv, lim);
-    uv = fminf(fmaxf(uv, -lim), lim);
-    const float y = gv / (1.f + expf(-a.alpha * gv)) * (uv + 1.f);
-    out[i] = x_from_f<E>(y * wt);
+    out[i] = x_from_f<E>(moe_gated(gv, uv, lim, a) * wt);
   }
 }
 
@@ -215,9 +250,7 @@ moe_sel_act_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w_gu, co
       float g = lane ? g1 : g0, u = lane ? u1 : u0;
       g = __bfloat162float(__float2bfloat16_rn(g));  // the projection's output is a bf16 row, as on the dense path
       u = __bfloat162float(__float2bfloat16_rn(u));
-      g = fminf(g, lim);
-      u = fminf(fmaxf(u, -lim), lim);
-      out[f + lane] = __float2bfloat16_rn(g / (1.f + expf(-a.alpha * g)) * (u + 1.f) * wt);
+      out[f + lane] = __float2bfloat16_rn(moe_gated(g, u, lim, a) * wt);
     }
   }
 }
@@ -270,7 +303,7 @@ extern "C" {
 
 int dli_moe_route(const float* h, const float* w_router, const float* correction, float* wts, float* idw, int32_t* sel_idx,
                   float* sel_w, int rows, int d, int n_out, int n_real, int top, int groups, int keep, float wscale,
-                  int renorm, dli_stream_t stream) {
+                  int renorm, const float* logit_bias, dli_stream_t stream) {
   DLI_CHECK_ARG(h && w_router && wts && idw && sel_idx && sel_w, "dli_moe_route: null pointer");
   if (groups < 1) groups = 1;
   DLI_CHECK_ARG(groups == 1 || (n_out % groups == 0 && keep >= 1 && keep <= groups && keep * (n_out / groups) >= top),
@@ -278,7 +311,7 @@ int dli_moe_route(const float* h, const float* w_router, const float* correction
   DLI_CHECK_ARG(d > 0 && n_out > 0 && n_real >= 0 && n_real <= n_out && top > 0 && top <= n_out && n_out <= 4096,
                 "dli_moe_route: %d router outputs (%d real experts), top %d", n_out, n_real, top);
   if (rows <= 0) return DLI_OK;
-  RouteArgs ra{w_router, correction, wts, idw, sel_idx, sel_w, n_out, n_real, top, groups, keep, wscale, renorm};
+  RouteArgs ra{w_router, correction, wts, idw, sel_idx, sel_w, n_out, n_real, top, groups, keep, wscale, renorm, logit_bias};
   DLI_LAUNCH("moe_route", moe_route_kernel, dim3(rows), dim3(rows <= 64 ? 512 : 256), (size_t)(2 * n_out + groups) * sizeof(float),
              static_cast<cudaStream_t>(stream), h, d, ra);
   return DLI_OK;
@@ -287,12 +320,12 @@ int dli_moe_route(const float* h, const float* w_router, const float* correction
 int dli_moe_act(const void* gu, const float* wts, void* act, int rows, int n_exp, int ff, float limit, int ff_s,
                 float limit_s, float alpha, int ld, int dt, int mode, dli_stream_t stream) {
   DLI_CHECK_ARG(gu && act && (wts || n_exp == 0) && n_exp >= 0 && ff >= 0 && ff_s >= 0 && n_exp * ff + ff_s > 0 &&
-                    (mode == 0 || mode == 1) && ld >= (mode == 1 ? 1 : 2) * (n_exp * ff + ff_s),
+                    mode >= 0 && mode <= 2 && ld >= (mode == 1 ? 1 : 2) * (n_exp * ff + ff_s),
                 "dli_moe_act: null pointer or bad shape");
   DLI_CHECK_ARG(dt == 0 || dt == 1, "element type %d: 0 = bf16, 1 = float", dt);
   if (rows <= 0) return DLI_OK;
   const int per = dt == 0 ? 8 : 4;
-  const int vec = mode == 1 && ff % per == 0 && ff_s % per == 0 && ld % per == 0 && aligned16(gu) && aligned16(act);
+  const int vec = mode >= 1 && ff % per == 0 && ff_s % per == 0 && ld % per == 0 && aligned16(gu) && aligned16(act);
   MoeAct a{n_exp, ff, limit, ff_s, limit_s, alpha, ld, mode, vec};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int work = (n_exp * ff + ff_s) / (vec ? per : 1);
@@ -309,7 +342,7 @@ int dli_moe_sel_supported(int d, int ff, int ff_s, int top) {
 int dli_moe_sel_bf16(const void* x, const void* w_gu, const void* w_down, const int32_t* sel_idx, const float* sel_w,
                      void* act_sel, void* y, int rows, int d, int n_exp, int top, int ff, float limit, int ff_s,
                      float limit_s, float alpha, int mode, dli_stream_t stream) {
-  DLI_CHECK_ARG(x && w_gu && w_down && sel_idx && sel_w && act_sel && y && (mode == 0 || mode == 1), "dli_moe_sel_bf16: null pointer");
+  DLI_CHECK_ARG(x && w_gu && w_down && sel_idx && sel_w && act_sel && y && mode >= 0 && mode <= 2, "dli_moe_sel_bf16: null pointer");
   DLI_CHECK_ARG(n_exp >= 0 && top >= 0 && dli_moe_sel_supported(d, ff, ff_s, top) && aligned16(w_gu) && aligned16(w_down),
                 "dli_moe_sel_bf16: sizes d=%d ff=%d ff_s=%d must be multiples of 8 and fit shared memory", d, ff, ff_s);
   if (rows <= 0) return DLI_OK;

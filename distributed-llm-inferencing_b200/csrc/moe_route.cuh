@@ -19,7 +19,8 @@ struct RouteArgs {
   int n_out, n_real, top;
   int groups, keep;       // groups > 1: only outputs of the `keep` best of that many equal groups can be chosen
   float wscale;
-  int renorm;             // 1: weights divided by the sum of the chosen scores
+  int renorm;             // 1: weights divided by the sum of the chosen scores (the softmax over the chosen logits alone)
+  const float* zb;        // [n_out] or NULL: added to the logits
 };
 
 // hr may have been written earlier in the same kernel (no __restrict__: plain coherent loads).
@@ -50,7 +51,7 @@ __device__ __forceinline__ void moe_route_row(const float* hr, int d, size_t row
       for (int c = lane; c < d; c += 32) acc = fmaf(hr[c], w[c], acc);
     }
     acc = warp_sum(acc);
-    if (lane == 0) zs[o] = acc;
+    if (lane == 0) zs[o] = acc + (ra.zb ? ra.zb[o] : 0.f);
   }
   __syncthreads();
   if (warp != 0) return;

@@ -212,7 +212,7 @@ int dli_layer_close(const void* y, const float* bias, const float* idw, const fl
                     float* tail, const int32_t* ent, float* out_f, void* out_e, int rows, int d, float eps, int dt,
                     const float* w_router, const float* correction, float* r_wts, float* r_idw, int32_t* r_sel_idx,
                     float* r_sel_w, int n_out, int n_real, int top, int groups, int keep, float wscale, int renorm,
-                    dli_stream_t stream) {
+                    const float* logit_bias, dli_stream_t stream) {
   DLI_CHECK_ARG(x && d > 0, "dli_layer_close: null pointer or empty shape");
   DLI_CHECK_ARG(y || !(bias || idw || ls), "dli_layer_close: bias, pass-through share and layer scale need a sublayer result");
   DLI_CHECK_ARG(!idw || h_in, "dli_layer_close: the pass-through share needs its input rows");
@@ -230,7 +230,7 @@ int dli_layer_close(const void* y, const float* bias, const float* idw, const fl
                 "%d groups of which %d are kept", n_out, n_real, top, groups, keep);
   if (rows <= 0) return DLI_OK;
   LayerClose a{bias, idw, h_in, ls, xs, xs_stride, n_prev, dwa, w_next, shift, tail, ent, out_f, eps, d, w_router ? 1 : 0,
-               RouteArgs{w_router, correction, r_wts, r_idw, r_sel_idx, r_sel_w, n_out, n_real, top, groups, keep, wscale, renorm}};
+               RouteArgs{w_router, correction, r_wts, r_idw, r_sel_idx, r_sel_w, n_out, n_real, top, groups, keep, wscale, renorm, logit_bias}};
   const size_t smem = w_router ? (size_t)(2 * n_out + groups) * sizeof(float) : 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   // 16-byte accesses when every row and vector starts on such a boundary

@@ -33,13 +33,21 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 
 // x[row] = table[ids[row]] * scale as fp32 (the residual stream starts in fp32).  With inv_freq [ceil(d/2)] a sinusoidal
 // position vector is added: channel 2i gets sin(p * inv_freq[i]), channel 2i+1 the cosine, p the row's position in its
-// sequence (from row_ent / ent), angle and functions in fp32.
+// sequence (from row_ent / ent), angle and functions in fp32.  With a pair table (BigramTab) the row of the hashed pair
+// (previous token, token) is added; x_copies > 1: the same row is also written to x + k * x_stride (several streams).
+struct BigramTab {
+  const void* table;        // [buckets + 1, d] or NULL; row `buckets` serves a sequence's first position
+  int buckets;
+  long long mul_prev, mul_cur;
+  int32_t* last;            // [slots]: the last token of the sequence in that slot
+};
+
 template <typename E>
 __global__ void __launch_bounds__(1024)
 embedding_f32_kernel(const int32_t* __restrict__ ids, const E* __restrict__ table, float* __restrict__ x,
                      float* __restrict__ x2, E* __restrict__ xe, int d, int vocab, float scale,
                      const int32_t* __restrict__ row_ent, const int32_t* __restrict__ ent,
-                     const float* __restrict__ inv_freq) {
+                     const float* __restrict__ inv_freq, BigramTab bg, int x_copies, size_t x_stride) {
   pdl_wait();
   pdl_trigger();
   const size_t row = blockIdx.x;
@@ -50,13 +58,33 @@ embedding_f32_kernel(const int32_t* __restrict__ ids, const E* __restrict__ tabl
     const int4 e = reinterpret_cast<const int4*>(ent)[row_ent[row]];
     pos = (float)(e.w + ((int)row - e.y));
   }
+  const E* brow = nullptr;
+  if (bg.table) {
+    // an entry's first row takes the previous token from the slot, and then (after every thread has read it) leaves the
+    // entry's last token there: no other CTA touches the slot
+    const int4 e = reinterpret_cast<const int4*>(ent)[row_ent[row]];  // slot, first row, rows, first position
+    const bool first = (int)row == e.y;
+    long long b = bg.buckets;
+    if (!(first && e.w == 0)) {
+      const long long prev = first ? bg.last[e.x] : ids[row - 1];
+      b = (prev * bg.mul_prev + (long long)ids[row] * bg.mul_cur) % bg.buckets;
+      if (b < 0) b += bg.buckets;
+    }
+    if (first) {
+      __syncthreads();
+      if (threadIdx.x == 0) bg.last[e.x] = ids[e.y + e.z - 1];
+    }
+    brow = reinterpret_cast<const E*>(bg.table) + (size_t)b * d;
+  }
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
     float v = to_f(table[(size_t)id * d + c]) * scale;
     if (inv_freq) {
       const float ang = pos * inv_freq[c >> 1];
       v += (c & 1) ? cosf(ang) : sinf(ang);
     }
+    if (brow) v += to_f(brow[c]);
     x[row * d + c] = v;
+    for (int k = 1; k < x_copies; ++k) x[k * x_stride + row * d + c] = v;
     if (x2) x2[row * d + c] = v;
     if (xe) xe[row * d + c] = from_f<E>(v);
   }
@@ -409,7 +437,7 @@ linear_any_kernel(const E* __restrict__ x, const E* __restrict__ w, O* __restric
 // act[m, f] = silu(gu[m, f] + b[f]) * (gu[m, F + f] + b[F + f]); bias [2F] fp32 or NULL
 template <typename E>
 __global__ void __launch_bounds__(256)
-silu_mul_kernel(const E* __restrict__ gu, E* __restrict__ act, int F, int ld, const float* __restrict__ bias, int vec) {
+silu_mul_kernel(const E* __restrict__ gu, E* __restrict__ act, int F, int ld, const float* __restrict__ bias, int vec, int act_fn) {
   pdl_wait();
   pdl_trigger();
   const size_t m = blockIdx.x;
@@ -429,7 +457,7 @@ silu_mul_kernel(const E* __restrict__ gu, E* __restrict__ act, int F, int ld, co
 #pragma unroll
       for (int k = 0; k < V; ++k) {
         if (bias) { g[k] += bias[f + k]; u[k] += bias[F + f + k]; }
-        o[k] = to_f(from_f<E>(silu_f(g[k]))) * u[k];
+        o[k] = act_fn ? gelu_new_f(g[k]) * u[k] : to_f(from_f<E>(silu_f(g[k]))) * u[k];
       }
       if constexpr (sizeof(E) == 2) st_16B(act + m * F + f, pack8(o));
       else *reinterpret_cast<float4*>(act + m * F + f) = make_float4(o[0], o[1], o[2], o[3]);
@@ -439,7 +467,7 @@ silu_mul_kernel(const E* __restrict__ gu, E* __restrict__ act, int F, int ld, co
   for (int f = blockIdx.y * blockDim.x + threadIdx.x; f < F; f += blockDim.x * gridDim.y) {
     float g = to_f(gu[m * ld + f]), u = to_f(gu[m * ld + F + f]);
     if (bias) { g += bias[f]; u += bias[F + f]; }
-    act[m * F + f] = from_f<E>(to_f(from_f<E>(silu_f(g))) * u);
+    act[m * F + f] = from_f<E>(act_fn ? gelu_new_f(g) * u : to_f(from_f<E>(silu_f(g))) * u);
   }
 }
 
@@ -574,15 +602,20 @@ extern "C" {
 
 int dli_embedding_f32(const int32_t* ids, const void* table, float* x, float* x2, void* xe, int rows, int d, int vocab,
                       float scale, int dt, const int32_t* row_ent, const int32_t* ent, const float* inv_freq,
-                      dli_stream_t stream) {
+                      const void* bigram, int buckets, long long mul_prev, long long mul_cur, int32_t* last, int x_copies,
+                      size_t x_stride, dli_stream_t stream) {
   DLI_CHECK_ARG(ids && table && x && d > 0 && vocab > 0, "dli_embedding_f32: null pointer or empty shape");
   DLI_CHECK_ARG(!inv_freq || (row_ent && ent && (reinterpret_cast<uintptr_t>(ent) & 15u) == 0),
                 "dli_embedding_f32: positions need row_ent and a 16-byte aligned ent");
+  DLI_CHECK_ARG(!bigram || (buckets > 0 && last && row_ent && ent && (reinterpret_cast<uintptr_t>(ent) & 15u) == 0),
+                "dli_embedding_f32: a pair table needs its row count, the slots' last tokens, row_ent and a 16-byte aligned ent");
+  DLI_CHECK_ARG(x_copies <= 1 || x_stride >= (size_t)rows * d, "dli_embedding_f32: copies of x overlap");
+  const BigramTab bg{bigram, buckets, mul_prev, mul_cur, last};
   DT_CHECK(dt);
   if (rows <= 0) return DLI_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dt == 0) DLI_LAUNCH("embedding_f32", embedding_f32_kernel<bf16>, dim3(rows), dim3(row_threads(rows, d)), 0, s, ids, (const bf16*)table, x, x2, (bf16*)xe, d, vocab, scale, row_ent, ent, inv_freq);
-  else DLI_LAUNCH("embedding_f32", embedding_f32_kernel<float>, dim3(rows), dim3(row_threads(rows, d)), 0, s, ids, (const float*)table, x, x2, (float*)xe, d, vocab, scale, row_ent, ent, inv_freq);
+  if (dt == 0) DLI_LAUNCH("embedding_f32", embedding_f32_kernel<bf16>, dim3(rows), dim3(row_threads(rows, d)), 0, s, ids, (const bf16*)table, x, x2, (bf16*)xe, d, vocab, scale, row_ent, ent, inv_freq, bg, x_copies, x_stride);
+  else DLI_LAUNCH("embedding_f32", embedding_f32_kernel<float>, dim3(rows), dim3(row_threads(rows, d)), 0, s, ids, (const float*)table, x, x2, (float*)xe, d, vocab, scale, row_ent, ent, inv_freq, bg, x_copies, x_stride);
   return DLI_OK;
 }
 
@@ -720,7 +753,8 @@ int dli_linear_any(const void* x, const void* w, void* y, int M, int N, int K, i
   return DLI_OK;
 }
 
-int dli_silu_mul(const void* gu, void* act, int M, int F, int ld, int dt, const float* bias, dli_stream_t stream) {
+int dli_silu_mul(const void* gu, void* act, int M, int F, int ld, int dt, const float* bias, int act_fn,
+                 dli_stream_t stream) {
   DLI_CHECK_ARG(gu && act && F > 0 && ld >= 2 * F, "dli_silu_mul: null pointer or bad shape");
   DT_CHECK(dt);
   if (M <= 0) return DLI_OK;
@@ -729,8 +763,8 @@ int dli_silu_mul(const void* gu, void* act, int M, int F, int ld, int dt, const 
   const int vec = F % per == 0 && ld % per == 0 && aligned16(gu) && aligned16(act);
   const int work = F / (vec ? per : 1);
   const dim3 grid(M, M <= 64 ? (work + 1023) / 1024 : (work >= 2048 ? 2 : 1));  // few or long rows: a row's channels go to several CTAs
-  if (dt == 0) DLI_LAUNCH("silu_mul", silu_mul_kernel<bf16>, grid, dim3(256), 0, s, (const bf16*)gu, (bf16*)act, F, ld, bias, vec);
-  else DLI_LAUNCH("silu_mul", silu_mul_kernel<float>, grid, dim3(256), 0, s, (const float*)gu, (float*)act, F, ld, bias, vec);
+  if (dt == 0) DLI_LAUNCH("silu_mul", silu_mul_kernel<bf16>, grid, dim3(256), 0, s, (const bf16*)gu, (bf16*)act, F, ld, bias, vec, act_fn);
+  else DLI_LAUNCH("silu_mul", silu_mul_kernel<float>, grid, dim3(256), 0, s, (const float*)gu, (float*)act, F, ld, bias, vec, act_fn);
   return DLI_OK;
 }
 

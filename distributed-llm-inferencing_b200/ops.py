@@ -477,20 +477,34 @@ def _f32(*ts):
         _req(t, torch.float32)
 
 
+def _cols(t, n, dtype=torch.bfloat16):
+    """A row-major matrix of n columns, or a range of n columns of one."""
+    if not t.is_cuda or t.dtype != dtype or t.dim() != 2 or t.shape[1] != n or t.stride(1) != 1:
+        raise ValueError(f"expected a CUDA {dtype} matrix of {n} columns with unit inner stride")
+
+
 def _i32(*ts):
     for t in ts:
         _req(t, torch.int32)
 
 
-def embedding_f32(ids, table, out, scale: float = 1.0, out2=None, out_e=None, row_ent=None, ent=None, inv_freq=None):
+def embedding_f32(ids, table, out, scale: float = 1.0, out2=None, out_e=None, row_ent=None, ent=None, inv_freq=None,
+                  bigram=None, mul_prev=0, mul_cur=0, last=None):
     """ids int32 [rows]; table [V, d] bf16 / float -> out float32 [rows, d] = table[ids] * scale (out2: a second copy;
     out_e: a copy in the table's element type).  inv_freq float32 [ceil(d/2)] with row_ent / ent: plus the sinusoidal
-    position vector (sin(p f_i) at channel 2i, cos(p f_i) at 2i+1)."""
-    _i32(ids, row_ent, ent), _req(table, table.dtype), _f32(out, out2, inv_freq), _req(out_e, table.dtype)
+    position vector (sin(p f_i) at channel 2i, cos(p f_i) at 2i+1).  bigram [n + 1, d] with row_ent / ent and last int32
+    [slots]: plus row (previous token * mul_prev + token * mul_cur) mod n, row n at position 0; last holds each slot's last
+    token and is advanced.  out [streams, >= rows, d]: the same rows go to every stream."""
+    _i32(ids, row_ent, ent, last), _req(table, table.dtype), _f32(out, out2, inv_freq), _req(out_e, table.dtype)
+    _req(bigram, table.dtype)
     if inv_freq is not None and inv_freq.numel() < (table.shape[1] + 1) // 2:
         raise ValueError("embedding_f32: one frequency per pair of channels")
+    copies, stride = (out.shape[0], out.stride(0)) if out.dim() == 3 else (1, 0)
+    if out.numel() // copies < ids.numel() * table.shape[1]:
+        raise ValueError("embedding_f32: output too small")
     _call("dli_embedding_f32", 1, _p(ids), _p(table), _p(out), _p(out2), _p(out_e), ids.numel(), table.shape[1],
-          table.shape[0], float(scale), _dt(table), _p(row_ent), _p(ent), _p(inv_freq), _stream())
+          table.shape[0], float(scale), _dt(table), _p(row_ent), _p(ent), _p(inv_freq), _p(bigram),
+          bigram.shape[0] - 1 if bigram is not None else 0, int(mul_prev), int(mul_cur), _p(last), copies, stride, _stream())
     return out
 
 
@@ -575,41 +589,45 @@ def linear_any(x, w, out):
     return out
 
 
-def silu_mul(gu, out, bias=None):
-    """out[m, f] = silu(gu[m, f] + b[f]) * (gu[m, F + f] + b[F + f]); bias float32 [2F] or None."""
+def silu_mul(gu, out, bias=None, gelu=False):
+    """out[m, f] = silu(gu[m, f] + b[f]) * (gu[m, F + f] + b[F + f]); bias float32 [2F] or None; gelu: the tanh form of gelu
+    instead of silu."""
     _req(gu, gu.dtype), _req(out, gu.dtype), _f32(bias)
-    _call("dli_silu_mul", 1, _p(gu), _p(out), gu.shape[0], out.shape[1], gu.shape[1], _dt(gu), _p(bias), _stream())
+    _call("dli_silu_mul", 1, _p(gu), _p(out), gu.shape[0], out.shape[1], gu.shape[1], _dt(gu), _p(bias), int(bool(gelu)), _stream())
     return out
 
 
 def attn_prep_append(proj, qbuf, k_cache, v_cache, row_ent, ent, page_table, H, G, D, V, rd, q_off, k_off, v_off,
-                     q_norm, k_norm, eps, cos_qk, sin_qk, cos_v, sin_v, bias=None, q_only=False):
+                     q_norm, k_norm, eps, cos_qk, sin_qk, cos_v, sin_v, bias=None, q_only=False, halves=False):
     """q/k head norms, rotation and value rotation of a ragged step; q -> qbuf (float32), k / v -> the paged caches.
     bias float32 (indexed like proj's columns) is added first; q_only: no keys or values are made or appended (the caches
-    are only asked for their page size)."""
+    are only asked for their page size).  halves: rotation pairs (i, i + rd/2) instead of (2i, 2i+1)."""
     _req(proj, proj.dtype), _req(k_cache, proj.dtype), _req(v_cache, proj.dtype)
     _f32(qbuf, q_norm, k_norm, cos_qk, sin_qk, cos_v, sin_v, bias), _i32(row_ent, ent, page_table)
     tl = cos_qk.shape[0] if cos_qk is not None else (cos_v.shape[0] if cos_v is not None else 0)
     _call("dli_attn_prep_append", 1, _p(proj), _p(qbuf), _p(k_cache), _p(v_cache), _p(row_ent), _p(ent), _p(page_table),
           page_table.shape[1], k_cache.shape[2], proj.shape[0], H, G, D, V, rd, proj.shape[1], q_off, k_off, v_off,
           _p(q_norm), _p(k_norm), float(eps), _p(cos_qk), _p(sin_qk), _p(cos_v), _p(sin_v), tl, _dt(proj), _p(bias),
-          1 if q_only else 0, _stream())
+          1 if q_only else 0, int(bool(halves)), _stream())
 
 
 def attn_ragged(qbuf, k_cache, v_cache, proj, out, row_ent, ent, page_table, H, G, D, V, scale, chunk=0, window=0,
-                sink=None, g_off=-1, cos_v=None, sin_v=None, ldv=0, splits=1, part=None, first=0, r1=None, r2=None):
+                sink=None, g_off=-1, cos_v=None, sin_v=None, ldv=0, splits=1, part=None, first=0, r1=None, r2=None, cap=0.0,
+                g_chan=False, out_scale=1.0):
     """Chunk- / window-masked attention with an optional sink and output gate over the paged cache -> out [rows, H*V].
     r1, r2 float32 [H]: the distance penalty r1 ln(1 + r2 (i - j)) on the scaled scores.
     first: positions below it stay visible whatever the chunk or window says.
     ldv: elements between value rows (0 = V); v_cache may be k_cache itself (values = leading part of the keys).
-    splits > 1: every row's keys are dealt to that many CTAs; part: float32 scratch of rows * H * splits * (V + 2)."""
-    _f32(qbuf, sink, cos_v, sin_v, part, r1, r2), _i32(row_ent, ent, page_table), _req(out, k_cache.dtype), _req(proj, k_cache.dtype)
+    splits > 1: every row's keys are dealt to that many CTAs; part: float32 scratch of rows * H * splits * (V + 2).
+    cap > 0: scores cap * tanh(score / cap); g_chan: one gate column per output channel; out_scale: a factor on the output;
+    out may be a column range of a wider row-major matrix."""
+    _f32(qbuf, sink, cos_v, sin_v, part, r1, r2), _i32(row_ent, ent, page_table), _cols(out, H * V, k_cache.dtype), _req(proj, k_cache.dtype)
     if splits > 1 and part.numel() < qbuf.shape[0] * H * splits * (V + 2):
         raise ValueError("attn_ragged: scratch too small for the key splits")
     _call("dli_attn_ragged", 2 if splits > 1 else 1, _p(qbuf), _p(k_cache), _p(v_cache), _p(proj), _p(out), _p(row_ent), _p(ent),
           _p(page_table), page_table.shape[1], k_cache.shape[2], qbuf.shape[0], H, G, D, V, float(scale), int(chunk),
           int(window), int(first), _p(sink), proj.shape[1] if proj is not None else 0, g_off, _p(cos_v), _p(sin_v), int(ldv),
-          int(splits), _p(part), _dt(k_cache), _p(r1), _p(r2), _stream())
+          int(splits), _p(part), _dt(k_cache), _p(r1), _p(r2), float(cap), int(bool(g_chan)), float(out_scale), out.stride(0), _stream())
     return out
 
 
@@ -618,17 +636,18 @@ def attn_ragged_tc_supported(D, V, dtype) -> bool:
 
 
 def attn_ragged_tc(qbuf, k_cache, v_cache, proj, out, ent, tiles, page_table, H, G, D, V, scale, chunk=0, window=0,
-                   sink=None, g_off=-1, cos_v=None, sin_v=None, page_base=0, first=0, r1=None, r2=None):
+                   sink=None, g_off=-1, cos_v=None, sin_v=None, page_base=0, first=0, r1=None, r2=None, cap=0.0, g_chan=False,
+                   out_scale=1.0):
     """attn_ragged for steps with portions of prompts, on the tensor cores: tiles int32 [n_tiles, 2] = (entry, first
     row of the 64-row query tile within the entry).  page_base: k_cache / v_cache hold pages page_base.. of the pool only
     (the pages the step's sequences use must all lie in that range)."""
-    _f32(qbuf, sink, cos_v, sin_v, r1, r2), _i32(ent, tiles, page_table), _req(out), _req(proj), _req(k_cache), _req(v_cache)
+    _f32(qbuf, sink, cos_v, sin_v, r1, r2), _i32(ent, tiles, page_table), _cols(out, H * V), _req(proj), _req(k_cache), _req(v_cache)
     kb = page_base * k_cache.stride(0) * k_cache.element_size()
     vb = page_base * v_cache.stride(0) * v_cache.element_size()
     _call("dli_attn_ragged_tc", 1, _p(qbuf), _p(k_cache) - kb, _p(v_cache) - vb, _p(proj), _p(out), _p(ent), _p(tiles),
           tiles.numel() // 2, _p(page_table), page_table.shape[1], k_cache.shape[2], H, G, D, V, float(scale), int(chunk),
           int(window), int(first), _p(sink), proj.shape[1] if proj is not None else 0, g_off, _p(cos_v), _p(sin_v), _p(r1),
-          _p(r2), _stream())
+          _p(r2), float(cap), int(bool(g_chan)), float(out_scale), out.stride(0), _stream())
     return out
 
 
@@ -760,22 +779,28 @@ def gated_group_rmsnorm(y, proj, w, out, groups, eps, z_off):
     return out
 
 
-def moe_route(h, w_router, correction, wts, idw, sel_idx, sel_w, n_real, top, groups=1, keep=1, wscale=1.0, renorm=True):
+def moe_route(h, w_router, correction, wts, idw, sel_idx, sel_w, n_real, top, groups=1, keep=1, wscale=1.0, renorm=True,
+              logit_bias=None):
     """Router of a mixture of experts on float32 rows: dense weights wts [rows, n_real], pass-through weight idw [rows],
     the choice sel_idx / sel_w [rows, top].  groups > 1: only outputs of the `keep` best of that many equal groups can be
-    chosen; renorm False: the weights are the scores themselves; both times wscale."""
-    _f32(h, w_router, correction, wts, idw, sel_w), _i32(sel_idx)
+    chosen; renorm False: the weights are the scores themselves; both times wscale.  logit_bias float32 [n_out]: added to
+    the logits (with renorm the weights are then the softmax over the chosen logits)."""
+    _f32(h, w_router, correction, wts, idw, sel_w, logit_bias), _i32(sel_idx)
     _call("dli_moe_route", 1, _p(h), _p(w_router), _p(correction), _p(wts), _p(idw), _p(sel_idx), _p(sel_w), h.shape[0],
           h.shape[1], w_router.shape[0], int(n_real), int(top), int(groups), int(keep), float(wscale), 1 if renorm else 0,
-          _stream())
+          _p(logit_bias), _stream())
 
 
-def moe_act(gu, wts, act, n_exp, ff, limit, ff_s=0, limit_s=0.0, alpha=1.702, gated=True):
+def _moe_mode(gated, silu):
+    return 1 if not gated else (2 if silu else 0)
+
+
+def moe_act(gu, wts, act, n_exp, ff, limit, ff_s=0, limit_s=0.0, alpha=1.702, gated=True, silu=False):
     """Activation of all experts' stacked projections, times the routing weights: the clamped gated form on [gate; up] rows,
-    or (gated False) max(u, 0)^2 on up rows alone."""
+    (silu) silu(g) * u on them, or (gated False) max(u, 0)^2 on up rows alone."""
     _req(gu, gu.dtype), _req(act, gu.dtype), _f32(wts)
     _call("dli_moe_act", 1, _p(gu), _p(wts), _p(act), gu.shape[0], int(n_exp), int(ff), float(limit), int(ff_s),
-          float(limit_s), float(alpha), gu.shape[1], _dt(gu), 0 if gated else 1, _stream())
+          float(limit_s), float(alpha), gu.shape[1], _dt(gu), _moe_mode(gated, silu), _stream())
     return act
 
 
@@ -783,12 +808,12 @@ def moe_sel_supported(d, ff, ff_s, top) -> bool:
     return bool(_lib.load().dli_moe_sel_supported(int(d), int(ff), int(ff_s), int(top)))
 
 
-def moe_sel(x, w_gu, w_down, sel_idx, sel_w, act_sel, y, n_exp, top, ff, limit, ff_s=0, limit_s=0.0, alpha=1.702, gated=True):
+def moe_sel(x, w_gu, w_down, sel_idx, sel_w, act_sel, y, n_exp, top, ff, limit, ff_s=0, limit_s=0.0, alpha=1.702, gated=True, silu=False):
     """Few rows (decode): the chosen experts' and the shared expert's weights only -> y [rows, d] (bf16)."""
     _req(x), _req(w_gu), _req(w_down), _req(act_sel), _req(y), _i32(sel_idx), _f32(sel_w)
     _call("dli_moe_sel_bf16", 2, _p(x), _p(w_gu), _p(w_down), _p(sel_idx), _p(sel_w), _p(act_sel), _p(y), x.shape[0],
-          x.shape[1], int(n_exp), int(top), int(ff), float(limit), int(ff_s), float(limit_s), float(alpha), 0 if gated else 1,
-          _stream())
+          x.shape[1], int(n_exp), int(top), int(ff), float(limit), int(ff_s), float(limit_s), float(alpha),
+          _moe_mode(gated, silu), _stream())
     return y
 
 
@@ -805,7 +830,7 @@ def layer_close(x, y=None, bias=None, idw=None, h_in=None, ls=None, xs=None, n_p
     _f32(x, bias, idw, h_in, ls, xs, dwa, w_next, shift, tail, out_f), _i32(ent)
     r = route or {}
     if route is not None:
-        _f32(r["w_router"], r.get("correction"), r["wts"], r["idw"], r["sel_w"]), _i32(r["sel_idx"])
+        _f32(r["w_router"], r.get("correction"), r.get("logit_bias"), r["wts"], r["idw"], r["sel_w"]), _i32(r["sel_idx"])
         if out_f is None or r["w_router"].shape[1] != x.shape[1]:
             raise ValueError("layer_close: the router reads the float32 normed rows")
     for t in (y, out_e):
@@ -819,7 +844,7 @@ def layer_close(x, y=None, bias=None, idw=None, h_in=None, ls=None, xs=None, n_p
           float(eps), _dt(ref) if ref is not None else 1, _p(r.get("w_router")), _p(r.get("correction")), _p(r.get("wts")),
           _p(r.get("idw")), _p(r.get("sel_idx")), _p(r.get("sel_w")), r["w_router"].shape[0] if route is not None else 0,
           int(r.get("n_real", 0)), int(r.get("top", 0)), int(r.get("groups", 1)), int(r.get("keep", 1)),
-          float(r.get("wscale", 1.0)), 1 if r.get("renorm", True) else 0, _stream())
+          float(r.get("wscale", 1.0)), 1 if r.get("renorm", True) else 0, _p(r.get("logit_bias")), _stream())
     return x
 
 
@@ -882,11 +907,69 @@ def delta_rule_ragged(qkv, proj, St, o, ent, H, G, D, V, b_off, a_off, a_log, dt
 
 
 def head_rmsnorm_gate(o, proj, w, out, H, V, eps, gate=1, g_off=0):
-    """out [rows, H*V] = o / rms_head(o) * w * act(proj[:, g_off + h*V + v]); w float32 [V] (shared) or [H*V];
-    gate 0 none, 1 SiLU, 2 sigmoid."""
-    _f32(o, w), _req(out, out.dtype)
+    """out [rows, H*V] = o / rms_head(o) * w * act(proj[:, g_off + h*V + v]); w float32 [V] (shared), [H*V] or None;
+    gate 0 none, 1 SiLU, 2 sigmoid.  out may be a column range of a wider row-major matrix."""
+    _f32(o, w), _cols(out, H * V, out.dtype)
     if proj is not None:
         _req(proj, out.dtype)
     _call("dli_head_rmsnorm_gate", 1, _p(o), _p(proj), _p(w), _p(out), o.shape[0], H, V, float(eps),
-          int(w.numel() == H * V and H > 1), int(gate), proj.shape[1] if proj is not None else 0, int(g_off), _dt(out), _stream())
+          int(w is not None and w.numel() == H * V and H > 1), int(gate), proj.shape[1] if proj is not None else 0, int(g_off),
+          out.stride(0), _dt(out), _stream())
     return out
+
+
+# ---------------------------------------------------------------------------------------------------------------
+# Several residual streams, linear attention (stream_rows.cu, linear_attn.cu)
+def streams_close(x, rows, y=None, mix=None, outw=None, in_next=None, w_next=None, out_f=None, out_e=None, eps: float = 1e-6,
+                  route=None):
+    """x float32 [streams, >= rows, d]: with y (the sublayer's result, element type) x_t <- sum_s mix[s, t] x_s + outw[t] y
+    in place; with w_next the norm of sum_s in_next[s] x_s (None: the plain sum) -> out_f (float32) / out_e (element type).
+    route: moe_route's arguments after h as a dict; the router runs on the normed row in the same kernel."""
+    _f32(x, mix, outw, in_next, w_next, out_f)
+    r = route or {}
+    if route is not None:
+        _f32(r["w_router"], r.get("correction"), r.get("logit_bias"), r["wts"], r["idw"], r["sel_w"]), _i32(r["sel_idx"])
+        if r["w_router"].shape[1] != x.shape[2]:
+            raise ValueError("streams_close: the router reads the normed rows")
+    for t in (y, out_e):
+        if t is not None:
+            _req(t, t.dtype)
+    if x.dim() != 3 or x.shape[1] < rows:
+        raise ValueError("streams_close: x [streams, >= rows, d]")
+    ref = y if y is not None else out_e
+    _call("dli_streams_close", 1, _p(y), _p(x), x.stride(0), x.shape[0], _p(mix), _p(outw), _p(in_next), _p(w_next), _p(out_f),
+          _p(out_e), int(rows), x.shape[2], float(eps), _dt(ref) if ref is not None else 1, _p(r.get("w_router")),
+          _p(r.get("logit_bias")), _p(r.get("correction")), _p(r.get("wts")), _p(r.get("idw")), _p(r.get("sel_idx")),
+          _p(r.get("sel_w")), r["w_router"].shape[0] if route is not None else 0, int(r.get("n_real", 0)), int(r.get("top", 0)),
+          int(r.get("groups", 1)), int(r.get("keep", 1)), float(r.get("wscale", 1.0)), 1 if r.get("renorm", True) else 0,
+          _stream())
+    return x
+
+
+def linattn_scratch_floats(n_tiles, H, D, V) -> int:
+    return int(_lib.load().dli_linattn_scratch_floats(int(n_tiles), int(H), int(D), int(V)))
+
+
+def linattn_ragged(proj, S, o, ent, H, D, V, q_off, k_off, v_off, silu=False, q_scale=1.0, k_scale=1.0, cos_t=None, sin_t=None,
+                   rd=0, log_decay=None, a_off=0, a2=None, a2_b=None, inv_tau=1.0, blocked=False, lg=None, tiles=None,
+                   scratch=None):
+    """Linear attention with a decaying matrix state over the rows of every entry; S float32 [slots, H, D, V] is advanced; o
+    float32 [rows, H*V].  log_decay float32 [H]: fixed decay per head; else a decay per key channel from columns a_off.. of
+    proj through a2 [H*D, rank], a2_b [H*D] (float32) and inv_tau.  blocked: small matrix products (steps with portions of
+    prompts; lg float32 scratch [rows, H*D] for a decay per channel), with tiles and scratch of linattn_scratch_floats(...)
+    floats the 64-row tiles of an entry in parallel."""
+    _req(proj, proj.dtype), _f32(S, o, cos_t, sin_t, log_decay, a2, a2_b, lg, scratch), _i32(ent, tiles)
+    rows, n_ent = proj.shape[0], ent.numel() // 4
+    n_tiles = tiles.numel() // 2 if tiles is not None else 0
+    gated = log_decay is None
+    par = bool(blocked) and scratch is not None and n_tiles > n_ent
+    if par and scratch.numel() < linattn_scratch_floats(n_tiles, H, D, V):
+        raise ValueError("linattn_ragged: scratch too small")
+    if o.numel() < rows * H * V or (gated and blocked and lg.numel() < rows * H * D):
+        raise ValueError("linattn_ragged: output or log-decay scratch too small")
+    _call("dli_linattn_ragged", (3 if par else 1) + int(gated and bool(blocked)), _p(proj), _p(S), _p(o), _p(ent), n_ent, rows, H, D,
+          V, proj.shape[1], int(q_off), int(k_off), int(v_off), int(bool(silu)), float(q_scale), float(k_scale), _p(cos_t),
+          _p(sin_t), int(rd), _p(log_decay), int(a_off), a2.shape[1] if a2 is not None else 0, _p(a2), _p(a2_b), float(inv_tau),
+          int(bool(blocked)), _p(lg), _p(tiles) if par else None, n_tiles if par else 0, _p(scratch) if par else None, _dt(proj),
+          _stream())
+    return o

@@ -2,13 +2,15 @@
 
 ShardEngine (engine.py) serves uniform Llama / GPT-2 stacks on rectangular batches with a bf16 residual stream.
 This engine serves stacks described layer by layer (HybridSpec): every layer has a token mixer — softmax attention
-with its options, latent attention, or a recurrent cell with a matrix state (mLSTM, state-space, gated delta rule) —
-and optionally a feed-forward (dense or a mixture of experts).  Four layer styles: sublayers in sequence, each
+with its options, latent attention, a recurrent cell with a matrix state (mLSTM, state-space, gated delta rule, linear
+attention with a fixed or an input-made decay), or two of these side by side on one input — and optionally a
+feed-forward (dense or a mixture of experts).  Five layer styles: sublayers in sequence, each
 wrapped in a pre-norm and a post-norm with one weight and reading its input through a short causal convolution;
 mixer and feed-forward side by side on one grouped norm; sublayers that read the residual stream itself and are
 normed on their output only, followed by a per-layer token input; pre-normed sublayers with a weight vector per
 norm, a layer scale on each result, a token shift in front of the mixer and an average over all layers' results
-after the layer.  Layers may share another layer's weights while
+after the layer; pre-normed sublayers that read a weighted sum of several residual streams and mix all of them
+afterwards.  Layers may share another layer's weights while
 keeping a cache / state of their own, or read another layer's cache.  The residual stream, norms, rotation
 angles, scores, softmax weights, convolution and recurrent state are fp32; projections run in the element type of the
 engine (bf16 on the tcgen05 / GEMV kernels of ops.linear, or float32 on the CUDA-core GEMM).
@@ -38,7 +40,8 @@ BF = torch.bfloat16
 
 @dataclass
 class MixerSpec:
-    kind: str                      # "attention", "mlstm", "latent_attention", "mamba2" or "delta"
+    kind: str                      # "attention", "mlstm", "latent_attention", "mamba2", "delta", "linear_attention" or
+                                   # "side_by_side" (the mixers in `parts` read one input, one projection sums their outputs)
     heads: int
     kv_heads: int
     dim: int                       # query / key size per head
@@ -74,6 +77,36 @@ class MixerSpec:
     # delta (gated delta rule): heads value heads of size vdim, kv_heads query/key heads of size dim, conv_taps of the
     # q / k / v convolution, scale on the unit queries, unit_eps under the root of the unit vectors
     unit_eps: float = 1e-6
+    # attention: soft cap of the scaled scores, a sink with score 0, values = the unrotated keys (no value projection)
+    softcap: float = 0.0
+    zero_sink: bool = False
+    keys_as_values: bool = False
+    # linear attention: S <- w S + k v^T, o = S^T q; w is `decay` (one per head), or per key channel sigmoid(low-rank
+    # projection)^(1/tau); factors on q and k, SiLU on q / k / v, one norm over all heads instead of one per head, the
+    # output gate's function
+    decay: Optional[tuple] = None
+    tau: float = 0.0
+    q_scale: float = 1.0
+    k_scale: float = 1.0
+    qkv_silu: bool = False
+    norm_heads_together: bool = False
+    gate_fn: str = "silu"          # or "sigmoid"
+    out_scale: float = 1.0         # factor on the mixer's output
+    parts: tuple = ()              # side_by_side: the MixerSpecs (one softmax attention, one linear attention)
+
+    @property
+    def flat(self) -> tuple:
+        return self.parts if self.kind == "side_by_side" else (self,)
+
+    @property
+    def out_width(self) -> int:
+        """Columns of the output projection's operand."""
+        return sum(m.heads * m.vdim for m in self.flat)
+
+    @property
+    def cached(self) -> Optional["MixerSpec"]:
+        """The part whose keys and values live in the paged cache."""
+        return next((m for m in self.flat if m.kind in ("attention", "latent_attention")), None)
 
 
 @dataclass
@@ -93,6 +126,8 @@ class MoESpec:
     keep: int = 1                  # can be chosen
     route_scale: float = 1.0       # factor on the routing weights
     renorm: bool = True            # weights divided by the sum of the chosen scores (False: the scores themselves)
+    act: str = "clamp"             # gated experts: the clamped form above, or "silu" (silu(g) * u)
+    router_bias: bool = False      # the router's logits have a bias
 
     @property
     def total_ff(self) -> int:
@@ -120,6 +155,7 @@ class LayerSpec:
     layer_scale: bool = False      # vectors ls1 / ls2 on the sublayers' results
     depth_avg: bool = False        # after the layer x <- sum_j dwa[j] X_j over the embedding output and all results so far
     ff_bias: bool = False          # the dense feed-forward's projections have biases
+    ff_fn: str = "silu"            # pre_norm: activation of the dense feed-forward's gate, or "gelu_tanh"
 
 
 @dataclass
@@ -136,6 +172,10 @@ class HybridSpec:
     side_width: int = 0            # > 0: columns of the side embedding table [vocab, side_width]
     pos_sinusoid: bool = False     # the embedding output gets sin / cos (position * pos_base^(-2i/width)) added
     pos_base: float = 10000.0
+    streams: int = 0               # > 0: that many residual streams (every layer pre_norm): a sublayer reads
+                                   # u = sum_s in[s] x_s, then x_t <- sum_s mix[s, t] x_s + out[t] * result
+    bigram: Optional[tuple] = None  # (buckets, mul_prev, mul_cur): a table row of the hashed pair (previous token, token) is
+                                   # added to the embedding
 
     @property
     def n_layers(self) -> int:
@@ -185,10 +225,10 @@ class RaggedEngine:
         self.is_first = self.is_last = self.has_head = True
         # layers that own a paged cache (a layer with kv_from reads its source's)
         self.attn_layers = [i for i, L in enumerate(spec.layers)
-                            if L.mixer.kind in ("attention", "latent_attention") and L.mixer.kv_from is None]
+                            if L.mixer.cached is not None and L.mixer.cached.kv_from is None]
         # latent attention caches ONE row [latent | rotated key part] per position and no values of its own
         shapes = [(1, m.kv_rank + m.rot_dims, 0) if m.kind == "latent_attention" else (m.kv_heads, m.dim, m.vdim)
-                  for m in (spec.layers[i].mixer for i in self.attn_layers)]
+                  for m in (spec.layers[i].mixer.cached for i in self.attn_layers)]
         self.kv = PagedKVCache(len(shapes), 0, 0, page_size, self.max_batch, self.max_seq_len, self.device,
                                pool_tokens=kv_pool_tokens, layer_shapes=shapes, dtype=dtype)
         self.kv_index = {li: n for n, li in enumerate(self.attn_layers)}
@@ -196,7 +236,14 @@ class RaggedEngine:
             if L.mixer.kv_from is not None:
                 self.kv_index[i] = self.kv_index[L.mixer.kv_from]
         self.slots = StateSlots(self.max_batch, self.device)
+        if spec.streams and not all(L.pre_norm and not (L.token_shift or L.layer_scale or L.depth_avg) for L in spec.layers):
+            raise ValueError("several residual streams: every layer pre-normed, without shift, layer scale or average")
+        if spec.bigram:
+            self.slots.add(("last",), dtype=torch.int32)       # the sequence's last token
         for i, L in enumerate(spec.layers):
+            for m in L.mixer.flat:
+                if m.kind == "linear_attention":
+                    self.slots.add(("S", i), m.heads, m.dim, m.vdim)
             if spec.taps > 1 and not L.post_only and not L.pre_norm:
                 self.slots.add(("tail1", i), spec.taps - 1, spec.width)
                 if L.ff:
@@ -280,6 +327,8 @@ class RaggedEngine:
 
         self.w = {"embed": t["embed"].to(E).contiguous().to(dev), "head": mat(t["head"]),
                   "final_norm": vec(t["final_norm"]) if s.norm_groups else float(t["final_norm"])}
+        if s.bigram:
+            self.w["bigram"] = t["bigram"].to(E).contiguous().to(dev)
         if s.side_width:
             self.w["side_embed"] = t["side_embed"].to(E).contiguous().to(dev)
         if s.loop_passes:
@@ -289,6 +338,38 @@ class RaggedEngine:
             # frequencies in float64 on the host, rounded once; the angle position * frequency is formed in fp32
             self.w["pos_freq"] = torch.tensor([s.pos_base ** (-2.0 * i / s.width) for i in range((s.width + 1) // 2)],
                                               dtype=torch.float64).to(torch.float32).to(dev)
+        def attention_rows(m, src, at):
+            """Projection rows q | k | (v) | (gate) of an attention mixer from column `at`, and its other tensors."""
+            qn, kn, vn = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
+            ws = [src["q"], src["k"]] + ([] if m.keys_as_values else [src["v"]]) + ([src["g"]] if m.head_gate or m.out_gate else [])
+            g = at + qn + kn + (0 if m.keys_as_values else vn)
+            # a norm without weights is the norm with unit weights; values that are the keys share their columns
+            ones = torch.ones(m.dim, dtype=torch.float32, device=dev)
+            sink = vec(src["sink"]) if m.sink else (torch.zeros(m.heads, dtype=torch.float32, device=dev) if m.zero_sink else None)
+            return ws, {"off": {"q": at, "k": at + qn, "v": at + qn + (0 if m.keys_as_values else kn),
+                                "g": g if m.head_gate or m.out_gate else -1},
+                        "qkv_b": vec(torch.cat([src[k].reshape(-1).float() for k in ("q_b", "k_b", "v_b")])) if m.bias else None,
+                        "q_norm": (vec(src["q_norm"]) if "q_norm" in src else ones) if m.qk_norm else None,
+                        "k_norm": (vec(src["k_norm"]) if "k_norm" in src else ones) if m.qk_norm else None, "sink": sink,
+                        "r1": vec(src["r1"]) if m.dist_penalty else None, "r2": vec(src["r2"]) if m.dist_penalty else None}
+
+        def linear_rows(m, src, at):
+            """Projection rows q | k | v | gate | (low-rank decay) of a linear-attention mixer from column `at`, and its other
+            tensors; a factor on the output goes into the norm's weight."""
+            hd, hv = m.heads * m.dim, m.heads * m.vdim
+            ws = [src["q"], src["k"], src["v"], src["g"]] + ([src["a1"]] if m.tau else [])
+            d = {"off": {"q": at, "k": at + hd, "v": at + 2 * hd, "g": at + 2 * hd + hv, "a": at + 2 * hd + 2 * hv}, "log_decay": None,
+                 "a2": None, "a2_b": None, "out_norm": vec(src["out_norm"]) if "out_norm" in src else None}
+            if m.tau:
+                d["a2"], d["a2_b"] = f32(src["a2"]), vec(src["a2_b"])
+            else:
+                # a decay of 0 keeps nothing: its logarithm is cut where the exponential is 0 anyway
+                d["log_decay"] = vec(torch.tensor([math.log(w) if w > 0 else -1e4 for w in m.decay], dtype=torch.float64).clamp(min=-1e4))
+            if m.out_scale != 1.0:
+                d["out_norm"] = (d["out_norm"] if d["out_norm"] is not None else
+                                 torch.ones(m.vdim, dtype=torch.float32, device=dev)) * m.out_scale
+            return ws, d
+
         self.layers = {}
         for i, src in t["layers"].items():
             L, m = s.layers[i], s.layers[i].mixer
@@ -308,15 +389,21 @@ class RaggedEngine:
                 d["qkv_b"] = vec(src["q_b"]) if m.bias else None
                 d["r1"], d["r2"] = (vec(src["r1"]), vec(src["r2"])) if m.dist_penalty else (None, None)
             elif m.kind == "attention":
-                d["w_proj"] = mat(src["q"], src["k"], src["v"], src["g"]) if m.head_gate else mat(src["q"], src["k"], src["v"])
-                d["off"] = {"q": 0, "k": qn, "v": qn + kn, "g": qn + kn + vn if m.head_gate else -1}
-                d["qkv_b"] = vec(torch.cat([src[k].reshape(-1).float() for k in ("q_b", "k_b", "v_b")])) if m.bias else None
-                # a norm without weights is the norm with unit weights
-                ones = torch.ones(m.dim, dtype=torch.float32, device=dev)
-                d["q_norm"] = (vec(src["q_norm"]) if "q_norm" in src else ones) if m.qk_norm else None
-                d["k_norm"] = (vec(src["k_norm"]) if "k_norm" in src else ones) if m.qk_norm else None
-                d["sink"] = vec(src["sink"]) if m.sink else None
-                d["r1"], d["r2"] = (vec(src["r1"]), vec(src["r2"])) if m.dist_penalty else (None, None)
+                ws, part = attention_rows(m, src, 0)
+                d["w_proj"] = mat(*ws)
+                d.update(part)
+            elif m.kind == "linear_attention":
+                ws, part = linear_rows(m, src, 0)
+                d["w_proj"] = mat(*ws)
+                d.update(part)
+            elif m.kind == "side_by_side":
+                rows_, d["parts"], at = [], [], 0
+                for pm, psrc in zip(m.parts, src["parts"]):
+                    ws, part = (linear_rows if pm.kind == "linear_attention" else attention_rows)(pm, psrc, at)
+                    rows_ += ws
+                    d["parts"].append(part)
+                    at += sum(w.shape[0] for w in ws)
+                d["w_proj"] = mat(*rows_)
             elif m.kind == "mlstm":
                 gn = m.heads * m.vdim
                 d["w_proj"] = mat(src["q"], src["k"], src["v"], src["g"], src["i"], src["f"])
@@ -361,7 +448,16 @@ class RaggedEngine:
                 d["a_log"], d["dt_bias"], d["out_norm"] = vec(src["A_log"]), vec(src["dt_bias"]), vec(src["out_norm"])
             else:
                 raise ValueError(f"layer {i}: mixer kind {m.kind!r}")
-            d["wo"] = mat(src["o"], pad_rows=False)
+            # mixers side by side share one output projection over their concatenated outputs
+            o_w = torch.cat([ps["o"] for ps in src["parts"]], dim=1) if m.kind == "side_by_side" else src["o"]
+            d["wo"] = mat(o_w, pad_rows=False)
+            if s.streams:
+                one = torch.ones(s.streams)
+                for n in ("hc1", "hc2") if (L.ff or L.moe is not None) else ("hc1",):
+                    if s.streams == 1 and n + "_in" not in src:   # one stream without weights: the plain residual sum
+                        d[n + "_in"], d[n + "_out"], d[n + "_mix"] = vec(one), vec(one), f32(torch.eye(1))
+                    else:
+                        d[n + "_in"], d[n + "_out"], d[n + "_mix"] = vec(src[n + "_in"]), vec(src[n + "_out"]), f32(src[n + "_mix"])
             if L.side_dim:
                 d["side_gate"], d["side_proj"] = mat(src["side_gate"], pad_rows=False), mat(src["side_proj"], pad_rows=False)
                 d["side_norm"] = vec(src["side_norm"])
@@ -380,6 +476,8 @@ class RaggedEngine:
                     d["w_gu"] = ops.pack_gate_up(src["gate"].to(BF), src["up"].to(BF)).to(dev)
                 else:
                     d["w_gu"] = mat(src["gate"], src["up"], pad_rows=False)
+                # {0, 0}: the epilogue's gelu form
+                d["ff_act"] = torch.zeros(2, dtype=torch.float32, device=dev) if L.ff_fn == "gelu_tanh" else None
                 d["gu_b"] = vec(torch.cat((src["gate_b"].reshape(-1).float(), src["up_b"].reshape(-1).float()))) if L.ff_bias else None
                 d["down_b"] = vec(src["down_b"]) if L.ff_bias else None
                 d["w_down"] = mat(src["down"], pad_rows=False)
@@ -415,7 +513,8 @@ class RaggedEngine:
                     downs.append(src["shared"][2])
                 d["w_gu"] = mat(*blocks)
                 d["w_down"] = torch.cat([x.to(E) for x in downs], dim=1).contiguous().to(dev)
-                d["w_router"], d["corr"] = f32(src["router"]), vec(src["correction"])
+                d["w_router"], d["corr"] = f32(src["router"]), vec(src["correction"]) if "correction" in src else None
+                d["router_b"] = vec(src["router_b"]) if e.router_bias else None
             self.layers[i] = d
 
     def weight_bytes(self) -> int:
@@ -455,9 +554,9 @@ class RaggedEngine:
             return
         s, dev, E = self.spec, self.device, self.dtype
         rows = _ceil(rows, 64)
-        mx = [L.mixer for L in s.layers]
+        mx = [m for L in s.layers for m in L.mixer.flat]
         n_proj = max(d["w_proj"].shape[0] for d in self.layers.values())
-        n_mix = max(m.heads * m.vdim for m in mx)
+        n_mix = max(L.mixer.out_width for L in s.layers)
         n_q = max([m.heads * m.dim for m in mx if m.kind == "attention"] +
                   [m.heads * (max(m.kv_rank, m.dim) + m.rot_dims) for m in mx if m.kind == "latent_attention"] + [1])
         ff = max([max(L.moe.total_ff, L.moe.top * L.moe.ff + L.moe.shared_ff) if L.moe is not None else L.ff
@@ -495,6 +594,11 @@ class RaggedEngine:
         if sides:
             self._sg = torch.empty(rows * max(sides), dtype=E, device=dev)
             self._sa = torch.empty(rows * max(sides), dtype=E, device=dev)
+        gated = [m.heads * m.dim for m in mx if m.kind == "linear_attention" and m.tau]
+        if gated:
+            self._lg = torch.empty(rows * max(gated), dtype=f32, device=dev)  # log decays per row and key channel
+        if s.streams:
+            self._xst = torch.empty(s.streams, rows, s.width, dtype=f32, device=dev)
         if any(L.parallel or L.pre_norm for L in s.layers):
             self._he = torch.empty(rows, s.width, dtype=E, device=dev)
             self._y2 = torch.empty(rows, s.width, dtype=E, device=dev)
@@ -656,6 +760,9 @@ class RaggedEngine:
         W = s.width
         x, hn, hc = self._x[:rows], self._hn[:rows], self._hc[:rows]
         y = self._y[:rows]
+        if s.streams:
+            self._stream_layers(rows, nw, views, long_step, tiles)
+            return self._head(self._hs[:rows], d_want, nw, logits_out)
         single = rows == n_ent and s.taps > 1 and self.layer_trace is None  # decode rows: norm + convolution fused
 
         def enter_sublayer(y_prev, g_post, g_next, tail, taps_w):
@@ -778,10 +885,15 @@ class RaggedEngine:
             ops.scalar_rmsnorm(x, self.w["final_norm"], s.eps, hn)
         else:
             ops.postnorm_add_norm(y_prev, x, g_prev, s.eps, hn, self.w["final_norm"])
+        return self._head(self._hs[:rows] if final_done else hn, d_want, nw, logits_out)
+
+    def _head(self, h, d_want, nw, logits_out):
+        """Logits of the wanted rows of the last norm's output h (None when no row is wanted)."""
         if nw == 0:
             return None
+        W, dev, E = self.spec.width, self.device, self.dtype
         hw = self._hw[:nw] if nw <= self._hw.shape[0] else torch.empty(nw, W, dtype=E, device=dev)
-        ops.gather_cast(self._hs[:rows] if final_done else hn, d_want, hw)
+        ops.gather_cast(h, d_want, hw)
         vp = self.w["head"].shape[0]
         logits = logits_out[:nw] if logits_out is not None else torch.empty(nw, vp, dtype=E, device=dev)
         self._lin(hw, self.w["head"], logits)
@@ -894,40 +1006,16 @@ class RaggedEngine:
         y_last = y
         if L.ff:
             ops.layer_close(x, y, ls=P["ls1"], w_next=P["norm2"], out_e=he, eps=s.eps)
-            act = self._act[:rows * L.ff].view(rows, L.ff)
-            if P["packed"] and 2 < rows <= 128 and s.width % 64 == 0:
-                ops.linear_splitk_gated_silu(he, P["w_gu"], self._splitk(), out=act)
-            elif P["packed"]:
-                ops.linear_gated_silu(he, P["w_gu"], out=act)
-            else:
-                gu = self._gu[:rows * 2 * L.ff].view(rows, 2 * L.ff)
-                self._lin(he, P["w_gu"], gu)
-                ops.silu_mul(gu, act, bias=P["gu_b"])
-            self._lin(act, P["w_down"], y)
+            self._dense_ff(L, P, he, y)
             close = {"ls": P["ls2"], "bias": P["down_b"]}
         elif L.moe is not None:
             e = L.moe
             y_last = self._y2[:rows]
-            wts = self._wts[:rows * e.experts].view(rows, e.experts)
-            idw = self._idw[:rows]
-            sel_idx, sel_w = self._sel_idx[:rows * e.top].view(rows, e.top), self._sel_w[:rows * e.top].view(rows, e.top)
+            route = self._route_args(e, P, rows)
+            idw = route["idw"]
             # the kernel that closes the mixer and norms the row also routes it
-            ops.layer_close(x, y, ls=P["ls1"], w_next=P["norm2"], out_f=hn, out_e=he, eps=s.eps,
-                            route=dict(w_router=P["w_router"], correction=P["corr"], wts=wts, idw=idw, sel_idx=sel_idx, sel_w=sel_w,
-                                       n_real=e.experts, top=e.top, groups=e.groups, keep=e.keep, wscale=e.route_scale,
-                                       renorm=e.renorm))
-            if self._moe_sel_ok(e, rows):
-                # decode rows of a sparse enough mixture: stream only the chosen experts' weights
-                n_sel = e.top * e.ff + e.shared_ff
-                ops.moe_sel(he, P["w_gu"], P["w_down"], sel_idx, sel_w, self._act[:rows * n_sel].view(rows, n_sel), y_last,
-                            e.experts, e.top, e.ff, e.limit, e.shared_ff, e.shared_limit, e.alpha, gated=e.gated)
-            else:
-                n_gu = P["w_gu"].shape[0]
-                gu = self._gu[:rows * n_gu].view(rows, n_gu)
-                self._lin(he, P["w_gu"], gu)
-                act = self._act[:rows * e.total_ff].view(rows, e.total_ff)
-                ops.moe_act(gu, wts, act, e.experts, e.ff, e.limit, e.shared_ff, e.shared_limit, e.alpha, gated=e.gated)
-                self._lin(act, P["w_down"], y_last)
+            ops.layer_close(x, y, ls=P["ls1"], w_next=P["norm2"], out_f=hn, out_e=he, eps=s.eps, route=route)
+            self._experts(e, P, he, route, y_last)
             close = {"ls": P["ls2"]}
             if e.identity:
                 close.update(idw=idw, h_in=hn)
@@ -941,6 +1029,123 @@ class RaggedEngine:
         else:
             ops.layer_close(x, y_last, eps=s.eps, **close)
 
+    def _dense_ff(self, L, P, he, y):
+        """y = down(act(gate he) * (up he)) without the down projection's bias; he, y [rows, width] in the element type."""
+        rows, W = he.shape
+        act = self._act[:rows * L.ff].view(rows, L.ff)
+        gelu = L.ff_fn == "gelu_tanh"
+        few = 2 < rows <= 128 and W % 64 == 0
+        if P["packed"] and gelu:
+            ops.linear_gated_act(he, P["w_gu"], P["ff_act"], self._splitk() if few else None, out=act)
+        elif P["packed"] and few:
+            ops.linear_splitk_gated_silu(he, P["w_gu"], self._splitk(), out=act)
+        elif P["packed"]:
+            ops.linear_gated_silu(he, P["w_gu"], out=act)
+        else:
+            gu = self._gu[:rows * 2 * L.ff].view(rows, 2 * L.ff)
+            self._lin(he, P["w_gu"], gu)
+            ops.silu_mul(gu, act, bias=P["gu_b"], gelu=gelu)
+        self._lin(act, P["w_down"], y)
+
+    def _route_args(self, e, P, rows):
+        """Arguments of the router for kernels that run it on a row they have just normed."""
+        return dict(w_router=P["w_router"], correction=P["corr"], logit_bias=P["router_b"],
+                    wts=self._wts[:rows * e.experts].view(rows, e.experts), idw=self._idw[:rows],
+                    sel_idx=self._sel_idx[:rows * e.top].view(rows, e.top), sel_w=self._sel_w[:rows * e.top].view(rows, e.top),
+                    n_real=e.experts, top=e.top, groups=e.groups, keep=e.keep, wscale=e.route_scale, renorm=e.renorm)
+
+    def _experts(self, e, P, he, route, y):
+        """y = the weighted sum of the chosen experts' (and the shared expert's) outputs for the rows he."""
+        rows = he.shape[0]
+        silu = e.act == "silu"
+        if self._moe_sel_ok(e, rows):
+            # decode rows of a sparse enough mixture: stream only the chosen experts' weights
+            n_sel = e.top * e.ff + e.shared_ff
+            ops.moe_sel(he, P["w_gu"], P["w_down"], route["sel_idx"], route["sel_w"], self._act[:rows * n_sel].view(rows, n_sel), y,
+                        e.experts, e.top, e.ff, e.limit, e.shared_ff, e.shared_limit, e.alpha, gated=e.gated, silu=silu)
+            return
+        n_gu = P["w_gu"].shape[0]
+        gu = self._gu[:rows * n_gu].view(rows, n_gu)
+        self._lin(he, P["w_gu"], gu)
+        act = self._act[:rows * e.total_ff].view(rows, e.total_ff)
+        ops.moe_act(gu, route["wts"], act, e.experts, e.ff, e.limit, e.shared_ff, e.shared_limit, e.alpha, gated=e.gated, silu=silu)
+        self._lin(act, P["w_down"], y)
+
+    # ------------------------------------------------------------------ layers with several residual streams
+    def _stream_layers(self, rows, nw, views, long_step, tiles):
+        """All layers of a model with several residual streams, from the embedding to the last norm (rows in _hs).  Between
+        two projections ONE kernel (ops.streams_close): the streams' mix with the sublayer's result, the next sublayer's
+        weighted sum of the streams, its norm and, in front of a mixture of experts, the router."""
+        s = self.spec
+        d_tok, d_rent, d_ent, d_want, d_tiles = views
+        xst, he, y = self._xst, self._he[:rows], self._y[:rows]
+        bg = s.bigram
+        ops.embedding_f32(d_tok, self.w["embed"], xst, s.embed_scale, row_ent=d_rent, ent=d_ent,
+                          bigram=self.w["bigram"] if bg else None, mul_prev=bg[1] if bg else 0, mul_cur=bg[2] if bg else 0,
+                          last=self.slots[("last",)] if bg else None)
+        P = self.layers[s.source(0)]
+        ops.streams_close(xst, rows, in_next=P["hc1_in"], w_next=P["norm1"], out_e=he, eps=s.eps)
+        for li, L in enumerate(s.layers):
+            P, m = self.layers[s.source(li)], L.mixer
+            n_proj, n_mix = P["w_proj"].shape[0], m.out_width
+            proj = self._proj[:rows * n_proj].view(rows, n_proj)
+            mix = self._mix[:rows * n_mix].view(rows, n_mix)
+            self._lin(he, P["w_proj"], proj)
+            at = 0
+            for pm, PP in zip(m.flat, P["parts"] if m.kind == "side_by_side" else (P,)):
+                out = mix[:, at:at + pm.heads * pm.vdim]
+                at += pm.heads * pm.vdim
+                if pm.kind == "attention":
+                    self._attention(li, pm, PP, proj, out, rows, views, tiles)
+                elif pm.kind == "linear_attention":
+                    self._linear_attention(li, pm, PP, proj, out, rows, views, long_step)
+                else:
+                    raise ValueError(f"layer {li}: mixer {pm.kind!r} has no form with several residual streams")
+            self._lin(mix, P["wo"], y)
+            last = li + 1 == s.n_layers
+            if last:
+                nxt = dict(w_next=self.w["final_norm"], out_f=self._hs[:rows]) if nw else {}
+            else:
+                Pn = self.layers[s.source(li + 1)]
+                nxt = dict(in_next=Pn["hc1_in"], w_next=Pn["norm1"], out_e=he)
+            hc = "hc1"
+            if L.ff or L.moe is not None:
+                route = self._route_args(L.moe, P, rows) if L.moe is not None else None
+                ops.streams_close(xst, rows, y, P["hc1_mix"], P["hc1_out"], P["hc2_in"], P["norm2"], out_e=he, eps=s.eps, route=route)
+                if L.moe is not None:
+                    self._experts(L.moe, P, he, route, y)
+                else:
+                    self._dense_ff(L, P, he, y)
+                hc = "hc2"
+            ops.streams_close(xst, rows, y, P[hc + "_mix"], P[hc + "_out"], eps=s.eps, **nxt)
+            if self.layer_trace is not None:
+                self.layer_trace.append(xst[:, :rows].sum(0))
+
+    def _linear_attention(self, li, m, P, proj, mix, rows, views, long_step):
+        """Linear attention with a decaying state: the recurrence over the state slot (row by row, or as small matrix
+        products for steps with portions of prompts), then the norm of the outputs and the gate."""
+        d_tok, d_rent, d_ent, d_want, d_tiles = views
+        off, H, D, V = P["off"], m.heads, m.dim, m.vdim
+        o = self._oscr[:rows * H * V].view(rows, H * V)
+        cos_t, sin_t = self._table(m.rot_base, m.rot_dims, m.rot_scaling) if m.rot_dims else (None, None)
+        scr, n_tiles, n_ent = None, d_tiles.numel() // 2, d_ent.numel() // 4
+        if long_step and n_tiles > n_ent and n_ent * H * ((V + 63) // 64) < 4 * self._sms:
+            # some entry spans several 64-row tiles and the (entry, head, 64 value columns) do not fill the GPU: all tiles at
+            # once (bounded scratch, else tiles in order)
+            need = ops.linattn_scratch_floats(n_tiles, H, D, V)
+            if need <= self.mlstm_parallel_max_floats:
+                if getattr(self, "_la_scr", None) is None or self._la_scr.numel() < need:
+                    self._la_scr = torch.empty(need, dtype=torch.float32, device=self.device)
+                scr = self._la_scr
+        ops.linattn_ragged(proj, self.slots[("S", li)], o, d_ent, H, D, V, off["q"], off["k"], off["v"], silu=m.qkv_silu,
+                           q_scale=m.q_scale, k_scale=m.k_scale, cos_t=cos_t, sin_t=sin_t, rd=m.rot_dims,
+                           log_decay=P["log_decay"], a_off=off["a"], a2=P["a2"], a2_b=P["a2_b"],
+                           inv_tau=1.0 / m.tau if m.tau else 1.0, blocked=long_step,
+                           lg=self._lg[:rows * H * D] if m.tau else None, tiles=d_tiles if scr is not None else None, scratch=scr)
+        n_h, n_v = (1, H * V) if m.norm_heads_together else (H, V)
+        ops.head_rmsnorm_gate(o, proj, P["out_norm"], mix, n_h, n_v, self.spec.eps, gate=1 if m.gate_fn == "silu" else 2,
+                              g_off=off["g"])
+
     def _attention(self, li, m, P, proj, mix, rows, views, tiles):
         """Softmax attention over the layer's paged keys and values: prep (head norms, rotation, append), then the
         tensor-core tiles for steps with portions of prompts where the sizes have one, else the row-wise kernel."""
@@ -952,13 +1157,14 @@ class RaggedEngine:
         cv, sv = self._table(m.rot_base, m.vdim, None) if m.rotate_values else (None, None)
         qbuf = self._qbuf[:rows * m.heads * m.dim].view(rows, m.heads * m.dim)
         r1, r2 = P.get("r1"), P.get("r2")
+        more = dict(cap=m.softcap, g_chan=m.out_gate, out_scale=m.out_scale)
         ops.attn_prep_append(proj, qbuf, kc, vc, d_rent, d_ent, pt, m.heads, m.kv_heads, m.dim, m.vdim,
                              m.rot_dims, off["q"], off["k"], off["v"], P["q_norm"], P["k_norm"], s.eps,
-                             cq, sq, cv, sv, bias=P.get("qkv_b"), q_only=m.kv_from is not None)
+                             cq, sq, cv, sv, bias=P.get("qkv_b"), q_only=m.kv_from is not None, halves=m.rot_halves)
         if tiles and m.scale > 0 and ops.attn_ragged_tc_supported(m.dim, m.vdim, E):
             ops.attn_ragged_tc(qbuf, kc, vc, proj, mix, d_ent, d_tiles, pt, m.heads, m.kv_heads, m.dim, m.vdim,
                                m.scale, chunk=m.chunk, window=m.window, sink=P["sink"], g_off=off["g"],
-                               cos_v=cv, sin_v=sv, first=m.keep_first, r1=r1, r2=r2)
+                               cos_v=cv, sin_v=sv, first=m.keep_first, r1=r1, r2=r2, **more)
         else:
             # few rows (decode): every row's keys go to several CTAs, so that a long context is read by many SMs; the
             # count depends on the rows alone (a replayed graph keeps it while the contexts grow).  A row never sees more
@@ -970,7 +1176,7 @@ class RaggedEngine:
             ops.attn_ragged(qbuf, kc, vc, proj, mix, d_rent, d_ent, pt, m.heads, m.kv_heads, m.dim, m.vdim,
                             m.scale, chunk=m.chunk, window=m.window, sink=P["sink"], g_off=off["g"], cos_v=cv,
                             sin_v=sv, first=m.keep_first, splits=splits, part=self._apart_att if splits > 1 else None,
-                            r1=r1, r2=r2)
+                            r1=r1, r2=r2, **more)
 
     def _delta(self, li, m, P, proj, mix, rows, views, long_step=False):
         """Gated delta rule: short convolutions and SiLU of q | k | v (fp32), the recurrence over the state slot, then
@@ -1019,24 +1225,10 @@ class RaggedEngine:
             return
         e = L.moe
         y2 = self._y2[:rows]
-        wts = self._wts[:rows * e.experts].view(rows, e.experts)
-        idw = self._idw[:rows]
-        ops.moe_route(hn, P["w_router"], P["corr"], wts, idw, self._sel_idx[:rows * e.top].view(rows, e.top),
-                      self._sel_w[:rows * e.top].view(rows, e.top), e.experts, e.top)
-        if self._moe_sel_ok(e, rows):
-            # decode rows of a sparse enough mixture: stream only the chosen experts' weights (and the shared expert's)
-            n_sel = e.top * e.ff + e.shared_ff
-            ops.moe_sel(he, P["w_gu"], P["w_down"], self._sel_idx[:rows * e.top].view(rows, e.top),
-                        self._sel_w[:rows * e.top].view(rows, e.top), self._act[:rows * n_sel].view(rows, n_sel), y2,
-                        e.experts, e.top, e.ff, e.limit, e.shared_ff, e.shared_limit, e.alpha)
-            ops.residual_add2(x, y, y2, idw if e.identity else None, hn if e.identity else None)
-            return
-        n_gu = P["w_gu"].shape[0]
-        gu = self._gu[:rows * n_gu].view(rows, n_gu)
-        self._lin(he, P["w_gu"], gu)
-        act = self._act[:rows * e.total_ff].view(rows, e.total_ff)
-        ops.moe_act(gu, wts, act, e.experts, e.ff, e.limit, e.shared_ff, e.shared_limit, e.alpha)
-        self._lin(act, P["w_down"], y2)
+        route = self._route_args(e, P, rows)
+        idw = route["idw"]
+        ops.moe_route(hn, **route)
+        self._experts(e, P, he, route, y2)
         ops.residual_add2(x, y, y2, idw if e.identity else None, hn if e.identity else None)
 
     def _moe_sel_ok(self, e, rows) -> bool:

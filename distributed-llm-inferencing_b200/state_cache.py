@@ -1,4 +1,4 @@
-"""Per-sequence state SLOTS: fixed-size fp32 state that a layer carries from token to token (the matrix memory
+"""Per-sequence state SLOTS: fixed-size state (fp32 unless stated) that a layer carries from token to token (the matrix memory
 of a recurrent layer, the last inputs of a short causal convolution), beside the paged key/value cache, which
 holds what grows with the sequence (engine.PagedKVCache; a slot's index is also its row of the page table).
 
@@ -21,9 +21,9 @@ class StateSlots:
         self.live: set = set()
         self.tensors: Dict[object, torch.Tensor] = {}
 
-    def add(self, key, *shape) -> torch.Tensor:
-        """Register float32 state of `shape` per slot under `key`; returns the [n_slots, *shape] tensor."""
-        t = torch.zeros(self.n_slots, *shape, dtype=torch.float32, device=self.device)
+    def add(self, key, *shape, dtype=torch.float32) -> torch.Tensor:
+        """Register state of `shape` per slot under `key`; returns the [n_slots, *shape] tensor."""
+        t = torch.zeros(self.n_slots, *shape, dtype=dtype, device=self.device)
         self.tensors[key] = t
         return t
 
@@ -43,4 +43,4 @@ class StateSlots:
             self.free.append(slot)
 
     def bytes(self) -> int:
-        return sum(t.numel() * 4 for t in self.tensors.values())
+        return sum(t.numel() * t.element_size() for t in self.tensors.values())

@@ -413,10 +413,14 @@ int dli_decode_advance(const int32_t* tokens, int32_t* token_log, int32_t* posit
 /* x = table[ids] * scale as fp32; x2 (optional) receives the same rows (a model that re-reads its embedding output),
  * xe (optional) the same rows in the element type (a first layer that reads the residual stream as a GEMM operand).
  * inv_freq [ceil(d/2)] fp32 (optional, with row_ent / ent): a sinusoidal position vector is added, channel 2i
- * sin(p * inv_freq[i]) and channel 2i+1 the cosine, p the row's position in its sequence (fp32 angles). */
+ * sin(p * inv_freq[i]) and channel 2i+1 the cosine, p the row's position in its sequence (fp32 angles).
+ * bigram [buckets + 1, d] in the element type (optional, with row_ent / ent): row (previous token * mul_prev + token *
+ * mul_cur) mod buckets is added, row `buckets` at position 0; last [slots] holds each slot's last token and is advanced.
+ * x_copies > 1: the rows also go to x + k * x_stride (models with several residual streams). */
 int dli_embedding_f32(const int32_t* ids, const void* table, float* x, float* x2, void* xe, int rows, int d, int vocab,
                       float scale, int dt, const int32_t* row_ent, const int32_t* ent, const float* inv_freq,
-                      dli_stream_t stream);
+                      const void* bigram, int buckets, long long mul_prev, long long mul_cur, int32_t* last, int x_copies,
+                      size_t x_stride, dli_stream_t stream);
 /* RMS norm in `groups` equal consecutive parts of the row, each by its own root mean square, times w [d] fp32;
  * hn (fp32) and he (element type dt) are optional outputs. */
 int dli_group_rmsnorm(const float* x, const float* w, float* hn, void* he, int rows, int d, int groups, float eps, int dt,
@@ -451,8 +455,9 @@ int dli_gather_cast(const float* src, const int32_t* rows, void* out, int n, int
 /* y[M,N] = x[M,K] . w[N,K]^T on the CUDA cores with fp32 accumulation: any shape, both element types. */
 int dli_linear_any(const void* x, const void* w, void* y, int M, int N, int K, int ldx, int ldy, int dt,
                    dli_stream_t stream);
-/* act[m, f] = silu(gu[m, f] + b[f]) * (gu[m, F + f] + b[F + f]); bias [2F] fp32 or NULL */
-int dli_silu_mul(const void* gu, void* act, int M, int F, int ld, int dt, const float* bias, dli_stream_t stream);
+/* act[m, f] = silu(gu[m, f] + b[f]) * (gu[m, F + f] + b[F + f]); bias [2F] fp32 or NULL; act_fn 1: gelu (tanh form) of the
+ * gate instead of silu */
+int dli_silu_mul(const void* gu, void* act, int M, int F, int ld, int dt, const float* bias, int act_fn, dli_stream_t stream);
 
 /* Attention of a ragged step.  dli_attn_prep_append: per-head RMS norm of q and k (q_norm / k_norm [D] fp32 or NULL),
  * rotation of the first rd dims (interleaved pairs; cos_qk / sin_qk [table_len, rd/2] fp32), rotation of the values
@@ -467,18 +472,21 @@ int dli_silu_mul(const void* gu, void* act, int M, int F, int ld, int dt, const 
  * through part [rows, H, splits, V + 2] fp32 and a merge kernel.
  * bias (dli_attn_prep_append, fp32, indexed like the columns of proj, or NULL) is added to the q / k / v columns first;
  * q_only != 0: only the queries are made, the layer reads another layer's cached keys and values.  r1 / r2 [H] fp32 (or
- * both NULL): the distance penalty r1[h] * ln(1 + r2[h] * (i - j)) is taken off the scaled score of query i, key j. */
+ * both NULL): the distance penalty r1[h] * ln(1 + r2[h] * (i - j)) is taken off the scaled score of query i, key j.
+ * halves: rotation pairs (i, i + rd/2) instead of (2i, 2i+1).  cap > 0: scaled scores become cap * tanh(score / cap).
+ * g_chan: the gate has a column per output channel, proj[row, g_off + h*V + v].  out_scale: a factor on the output.  ldo:
+ * elements between output rows (0 = H*V), for outputs that are a part of wider rows. */
 int dli_attn_prep_append(const void* proj, float* qbuf, void* k_cache, void* v_cache, const int32_t* row_ent,
                          const int32_t* ent, const int32_t* page_table, int max_pages, int page_size, int rows, int H,
                          int G, int D, int V, int rd, int ldp, int q_off, int k_off, int v_off, const float* q_norm,
                          const float* k_norm, float eps, const float* cos_qk, const float* sin_qk, const float* cos_v,
-                         const float* sin_v, int table_len, int dt, const float* bias, int q_only, dli_stream_t stream);
+                         const float* sin_v, int table_len, int dt, const float* bias, int q_only, int halves,
+                         dli_stream_t stream);
 int dli_attn_ragged(const float* qbuf, const void* k_cache, const void* v_cache, const void* proj, void* out,
                     const int32_t* row_ent, const int32_t* ent, const int32_t* page_table, int max_pages, int page_size,
                     int rows, int H, int G, int D, int V, float scale, int chunk, int window, int first, const float* sink,
                     int ldp, int g_off, const float* cos_v, const float* sin_v, int ldv, int splits, float* part, int dt,
-                    const float* r1, const float* r2,
-                    dli_stream_t stream);
+                    const float* r1, const float* r2, float cap, int g_chan, float out_scale, int ldo, dli_stream_t stream);
 
 /* The same attention for steps that hold portions of prompts, on the tensor cores (bf16 caches only): one CTA per
  * 64-row query tile of an entry and query head; tiles[2t] = entry, tiles[2t+1] = first row of the tile within the
@@ -488,7 +496,7 @@ int dli_attn_ragged_tc(const float* qbuf, const void* k_cache, const void* v_cac
                        const int32_t* ent, const int32_t* tiles, int n_tiles, const int32_t* page_table, int max_pages,
                        int page_size, int H, int G, int D, int V, float scale, int chunk, int window, int first,
                        const float* sink, int ldp, int g_off, const float* cos_v, const float* sin_v, const float* r1,
-                       const float* r2, dli_stream_t stream);
+                       const float* r2, float cap, int g_chan, float out_scale, int ldo, dli_stream_t stream);
 
 /* Matrix-memory recurrent layer (mLSTM, stabilised): q, k, v, gate pre-activations and the output gate are columns
  * of proj [rows, ldp]; state S [slots, H, D, V], n [slots, H, D], m [slots, H] fp32 is read and advanced (an entry
@@ -567,10 +575,12 @@ int dli_gated_group_rmsnorm(const float* y, const void* proj, const float* w, vo
 /* groups > 1: the n_out outputs form that many equal groups of neighbours, a group's score is its largest score +
  * correction, and only outputs of the `keep` best groups can be chosen.  renorm 0: the weights are the scores
  * themselves; both forms times wscale.  mode 1 (dli_moe_act, dli_moe_sel_bf16): experts without a gate,
- * act = max(u, 0)^2 * weight on gu [rows, ld] = the experts' stacked up projections [ff each], then the shared one's. */
+ * act = max(u, 0)^2 * weight on gu [rows, ld] = the experts' stacked up projections [ff each], then the shared one's.
+ * mode 2: silu(g) * u * weight, no limits.  logit_bias [n_out] or NULL is added to the logits; with renorm 1 the weights
+ * are then the softmax over the chosen logits alone. */
 int dli_moe_route(const float* h, const float* w_router, const float* correction, float* wts, float* idw, int32_t* sel_idx,
                   float* sel_w, int rows, int d, int n_out, int n_real, int top, int groups, int keep, float wscale,
-                  int renorm, dli_stream_t stream);
+                  int renorm, const float* logit_bias, dli_stream_t stream);
 int dli_moe_act(const void* gu, const float* wts, void* act, int rows, int n_exp, int ff, float limit, int ff_s,
                 float limit_s, float alpha, int ld, int dt, int mode, dli_stream_t stream);
 /* Few rows (decode steps, bf16): only the weights of each row's chosen experts (and the shared expert) are read.
@@ -597,7 +607,7 @@ int dli_layer_close(const void* y, const float* bias, const float* idw, const fl
                     float* tail, const int32_t* ent, float* out_f, void* out_e, int rows, int d, float eps, int dt,
                     const float* w_router, const float* correction, float* r_wts, float* r_idw, int32_t* r_sel_idx,
                     float* r_sel_w, int n_out, int n_real, int top, int groups, int keep, float wscale, int renorm,
-                    dli_stream_t stream);
+                    const float* logit_bias, dli_stream_t stream);
 int dli_token_shift_ragged(const float* h, const float* shift, float* tail, const int32_t* row_ent, const int32_t* ent,
                            void* out, int rows, int d, int dt, dli_stream_t stream);
 
@@ -631,7 +641,33 @@ int dli_delta_rule_ragged(const float* qkv, const void* proj, float* St, float* 
                           int G, int D, int V, int ldx, int ldp, int b_off, int a_off, const float* a_log,
                           const float* dt_bias, float q_scale, float unit_eps, int blocked, int dt, dli_stream_t stream);
 int dli_head_rmsnorm_gate(const float* o, const void* proj, const float* w, void* out, int rows, int H, int V, float eps,
-                          int w_heads, int gate, int ldp, int g_off, int dt, dli_stream_t stream);
+                          int w_heads, int gate, int ldp, int g_off, int ldo, int dt, dli_stream_t stream);
+
+/* Layers with several residual streams (hyper-connections): x holds n_streams (1..8) fp32 streams, stream t at
+ * x + t * xs_stride.  With y (element type) x_t <- sum_s mix[s, t] x_s + outw[t] y, all from the old streams; with w_next
+ * u = sum_s in_next[s] x_s (in_next NULL: the plain sum) is normed, rmsnorm(u) * w_next -> out_f (fp32) / out_e (element
+ * type), either may be NULL; with w_router the router of a mixture of experts runs on that row (arguments as in
+ * dli_moe_route). */
+int dli_streams_close(const void* y, float* x, size_t xs_stride, int n_streams, const float* mix, const float* outw,
+                      const float* in_next, const float* w_next, float* out_f, void* out_e, int rows, int d, float eps, int dt,
+                      const float* w_router, const float* logit_bias, const float* correction, float* r_wts, float* r_idw,
+                      int32_t* r_sel_idx, float* r_sel_w, int n_out, int n_real, int top, int groups, int keep, float wscale,
+                      int renorm, dli_stream_t stream);
+
+/* Linear attention with a decaying matrix state: S_t = diag(w_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head, S
+ * [slots, H, D, V] fp32 read and advanced (an entry at position 0 starts from zero), o [rows, H*V] fp32.  q, k [H, D] and
+ * v [H, V] are columns of proj [rows, ldp]; silu != 0: SiLU on all three; rd > 0: the first rd dimensions of q and k are
+ * rotated in pairs (i, i + rd/2) (cos_t / sin_t [positions, rd/2]); q_scale / k_scale: factors.  The decay is
+ * exp(log_decay[h]), or, with log_decay NULL, per key channel sigmoid(a2 . proj[row, a_off : +rank] + a2_b)^inv_tau
+ * (a2 [H*D, rank], a2_b [H*D] fp32).  blocked != 0 (steps with portions of prompts): 16 rows at a time as small matrix
+ * products, else row by row; lg: scratch [rows, H*D] for the blocked form with a decay per channel; with tiles (as for
+ * dli_attn_ragged_tc) and scratch of dli_linattn_scratch_floats floats the 64-row tiles of an entry run in parallel. */
+size_t dli_linattn_scratch_floats(int n_tiles, int H, int D, int V);
+int dli_linattn_ragged(const void* proj, float* S, float* o, const int32_t* ent, int n_ent, int rows, int H, int D, int V, int ldp,
+                       int q_off, int k_off, int v_off, int silu, float q_scale, float k_scale, const float* cos_t,
+                       const float* sin_t, int rd, const float* log_decay, int a_off, int rank, const float* a2, const float* a2_b,
+                       float inv_tau, int blocked, float* lg, const int32_t* tiles, int n_tiles, float* scratch, int dt,
+                       dli_stream_t stream);
 
 #ifdef __cplusplus
 }
