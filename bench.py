@@ -1075,6 +1075,190 @@ def gimudra_kernel_times(eng, spec, T, peaks):
     return res
 
 
+# ---------------------------------------------------------------------------------- Salizen beside Togalorn and Gimudra
+def salizen_config(width, heads, kv, hd, ff, layers, vocab, window=512):
+    """The Salizen design at the sizes of a Llama layer, two residual streams: lightning attention with the Llama layer's
+    head count and head size and the dense feed-forward, the same with a mixture of 16 experts of size ff/4 (4 per token),
+    windowed attention with the Llama layer's heads beside gated linear attention with half as many (dense), retention
+    (mixture); repeated."""
+    decay = [1.0 - 2.0 ** (-5.0 - 3.0 * h / heads) for h in range(heads)]
+    lin = {"heads": heads, "dim": hd, "vdim": hd, "decay": decay}
+    par = {"left_scale": 0.6, "right_scale": 0.5,
+           "left": {"heads": heads, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 30.0, "mask": {"size": window},
+                    "rot": {"base": 500000.0, "dims": hd // 2, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+           "right": {"heads": heads // 2, "dim": hd, "vdim": hd, "tau": 16.0}}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 16, "top": 4}}
+    kinds = [("lightning", lin, dense), ("lightning", lin, moe), ("parallel", par, dense),
+             ("retention", dict(lin, rot={"base": 10000.0, "dims": hd}), moe)]
+    return {"architecture": "Salizen", "vocab": vocab, "width": width, "streams": 2, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 30011, "mul_prev": 31, "mul_cur": 7}},
+            "layers": [dict(zip(("type", "mixer", "mlp"), kinds[i % 4])) for i in range(layers)]}
+
+
+def run_salizen_compare(args, peaks):
+    """Prefill and decode throughput of the Salizen design beside the framework's closest models on RaggedEngine — the
+    Togalorn design (a recurrence with a matrix state, gated experts) and the Gimudra design (pre-normed layers closed by
+    one kernel, masked attention, experts) — at equal layer sizes and depth, random weights, plus each kernel of the new
+    mechanisms alone against its roofline.  One JSON line; the default workload of this file is untouched."""
+    from dli_b200 import gimudra, salizen, togalorn
+    from dli_b200.ragged_engine import RaggedEngine
+
+    T, K, W = args.ctx, args.steps, args.warmup
+    out = {"metric": "salizen_vs_togalorn_gimudra", "unit": "tokens/s", "ctx": T, "steps": K, "warmup": W, "dtype": "bf16",
+           "data": "synthetic", "peaks": peaks, "sizes": {}}
+    names = args.hybrid_sizes.split(",")
+    if len(names) > 1:
+        import subprocess
+        for name in names:
+            cmd = [sys.executable, os.path.abspath(__file__), "--compare-salizen", "--hybrid-sizes", name, "--steps", str(K),
+                   "--warmup", str(W), "--ctx", str(T), "--batch", str(args.batch), "--page-size", str(args.page_size)]
+            p = subprocess.run(cmd, capture_output=True, text=True, check=True)
+            out["sizes"].update(json.loads(p.stdout.strip().splitlines()[-1])["sizes"])
+        return out
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    for name in names:
+        width, heads, kv, hd, ff, layers, vocab = HYBRID_SIZES[name]
+        mods = ((salizen, salizen_config(width, heads, kv, hd, ff, layers, vocab), "salizen"),
+                (togalorn, togalorn_config(width, heads, kv, hd, ff, layers, vocab), "togalorn"),
+                (gimudra, gimudra_config(width, heads, kv, hd, ff, layers, vocab), "gimudra"))
+        res = {}
+        for mod, cfg, tag in mods:
+            spec = mod.spec_from_config(cfg)
+            eng = RaggedEngine(spec, max_batch=max(args.batch, 8), max_seq_len=T + K + W + 64, page_size=args.page_size)
+            eng.load_tensors(mod.model_tensors(spec, mod.random_state_dict(spec, seed=1, std=0.02, device="cuda")))
+            res.update(ragged_throughput(eng, vocab, T, K, W, args.batch, tag, flush))
+            res[f"{tag}_kernels"] = {"salizen": salizen_kernel_times, "togalorn": togalorn_kernel_times,
+                                     "gimudra": gimudra_kernel_times}[tag](eng, spec, T, peaks)
+            eng.unload()
+            del eng
+            torch.cuda.empty_cache()
+        out["sizes"][name] = res
+    return out
+
+
+def salizen_kernel_times(eng, spec, T, peaks):
+    """Each kernel of the Salizen mechanisms alone at the step sizes of the comparison: a T-token portion (prefill) and
+    the prompt's last token alone (decode), against its algorithmic HBM bytes or FLOPs and the measured peaks (fp32: the
+    nominal CUDA-core rate at the maximum clock)."""
+    from dli_b200 import ops
+
+    dev, E, W = eng.device, eng.dtype, spec.width
+    hbm, tc = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    fp32 = 2.0 * 128 * eng._sms * peaks.get("sm_max_mhz", 1965.0) * 1e6
+    res = {}
+
+    def timeit(fn, n=5, reps=10):
+        fn()
+        return statistics.median(ev_time_ms(lambda: [fn() for _ in range(reps)]) for _ in range(n)) / reps
+
+    def put(key, ms, byt=None, flops=None, cuda_core=None):
+        d = {"ms": round(ms, 4)}
+        if byt is not None:
+            d["of_hbm"] = round(byt / (ms / 1e3) / hbm, 3)
+        if flops is not None:
+            d["of_bf16_peak"] = round(flops / (ms / 1e3) / tc, 4)
+        if cuda_core is not None:
+            d["of_fp32_peak"] = round(cuda_core / (ms / 1e3) / fp32, 4)
+        res[key] = d
+
+    slot = eng.open_sequence()
+    eng.kv.reserve(slot, T + 1)
+    eng.kv.commit()
+    S, eb = spec.streams, 2
+    for tag, rows, start in (("prefill", T, 0), ("decode", 1, T - 1)):
+        eng._workspace(rows)
+        row_ent = torch.zeros(rows, dtype=torch.int32, device=dev)
+        ent = torch.tensor([slot, 0, rows, start], dtype=torch.int32, device=dev)
+        d_tiles = torch.tensor([[0, q0] for q0 in range(0, rows, 64)] if rows > 1 else [], dtype=torch.int32, device=dev).flatten()
+        views = (None, row_ent, ent, None, d_tiles)
+        x = torch.randn(S, rows, W, device=dev)
+        he = torch.empty(rows, W, dtype=E, device=dev)
+        y = torch.randn(rows, W, device=dev).to(E)
+        ids = torch.randint(0, spec.vocab, (rows,), dtype=torch.int32, device=dev)
+        put(f"{tag}_embedding_bigram", timeit(lambda: ops.embedding_f32(ids, eng.w["embed"], x, 1.0, row_ent=row_ent, ent=ent,
+                                                                         bigram=eng.w["bigram"], mul_prev=31, mul_cur=7,
+                                                                         last=eng.slots[("last",)])), byt=rows * W * (2 * eb + 4 * S))
+        li_m = next(i for i, L in enumerate(spec.layers) if L.moe is not None)
+        P, e = eng.layers[li_m], spec.layers[li_m].moe
+        byt = rows * W * (8 * S + 2 * eb)
+        put(f"{tag}_streams_close_norm", timeit(lambda: ops.streams_close(x, rows, y, P["hc1_mix"], P["hc1_out"], P["hc2_in"], P["norm2"],
+                                                                          out_e=he, eps=1e-6)), byt=byt)
+        route = eng._route_args(e, P, rows)
+        put(f"{tag}_streams_close_norm_route", timeit(lambda: ops.streams_close(x, rows, y, P["hc1_mix"], P["hc1_out"], P["hc2_in"],
+                                                                                P["norm2"], out_e=he, eps=1e-6, route=route)),
+            byt=byt + P["w_router"].numel() * 4)
+        x.normal_()
+        # linear attention: lightning, retention, gated (beside softmax attention)
+        for name, want in (("lightning", lambda m: m.qkv_silu), ("retention", lambda m: m.decay and not m.qkv_silu), ("gated", lambda m: m.tau)):
+            li, m, PP = next((i, m, (eng.layers[i]["parts"][k] if L.mixer.kind == "side_by_side" else eng.layers[i]))
+                             for i, L in enumerate(spec.layers) for k, m in enumerate(L.mixer.flat)
+                             if m.kind == "linear_attention" and want(m))
+            H, D, V = m.heads, m.dim, m.vdim
+            proj = (0.5 * torch.randn(rows, eng.layers[li]["w_proj"].shape[0], device=dev)).to(E)
+            mix = torch.empty(rows, H * V, dtype=E, device=dev)
+            ms = timeit(lambda: eng._linear_attention(li, m, PP, proj, mix, rows, views, rows > 1), n=3, reps=5)
+            o = torch.randn(rows, H * V, device=dev)
+            nh, nv = (1, H * V) if m.norm_heads_together else (H, V)
+            ms_n = timeit(lambda: ops.head_rmsnorm_gate(o, proj, PP["out_norm"], mix, nh, nv, 1e-6, gate=1, g_off=PP["off"]["g"]))
+            put(f"{tag}_{name}_norm_gate", ms_n, byt=rows * H * V * (4 + 2 * eb))
+            if rows > 1:
+                put(f"{tag}_{name}_recurrence", ms - ms_n, cuda_core=4 * rows * H * D * V)   # update and read-out of the state
+                res[f"{tag}_{name}_recurrence"]["of_hbm"] = round(rows * H * (2 * D * eb + V * (eb + 4)) / ((ms - ms_n) / 1e3) / hbm, 3)
+            else:
+                put(f"{tag}_{name}_recurrence", ms - ms_n, byt=2 * H * D * V * 4)
+        # windowed attention with soft cap, sink and a gate per channel; without the cap
+        li = next(i for i, L in enumerate(spec.layers) if L.mixer.kind == "side_by_side")
+        m, PP = spec.layers[li].mixer.parts[0], eng.layers[li]["parts"][0]
+        proj = (0.5 * torch.randn(rows, eng.layers[li]["w_proj"].shape[0], device=dev)).to(E)
+        mix = torch.empty(rows, m.heads * m.vdim, dtype=E, device=dev)
+        qbuf = torch.empty(rows, m.heads * m.dim, device=dev)
+        kc, vc = eng.kv.k[eng.kv_index[li]], eng.kv.v[eng.kv_index[li]]
+        cos_t, sin_t = eng._table(m.rot_base, m.rot_dims, m.rot_scaling)
+        off, win = PP["off"], m.window or T
+        put(f"{tag}_attn_prep", timeit(lambda: ops.attn_prep_append(proj, qbuf, kc, vc, row_ent, ent, eng.kv.page_table, m.heads,
+                                                                     m.kv_heads, m.dim, m.vdim, m.rot_dims, off["q"], off["k"], off["v"],
+                                                                     None, None, 1e-6, cos_t, sin_t, None, None, halves=True)))
+        for cap in (m.softcap, 0.0):
+            key = f"{tag}_attn" + ("" if cap else "_without_cap")
+            kw = dict(window=m.window, sink=PP["sink"], g_off=off["g"], cap=cap, g_chan=True, out_scale=m.out_scale)
+            if rows > 1 and ops.attn_ragged_tc_supported(m.dim, m.vdim, E):
+                ms = timeit(lambda: ops.attn_ragged_tc(qbuf, kc, vc, proj, mix, ent, d_tiles, eng.kv.page_table, m.heads, m.kv_heads,
+                                                       m.dim, m.vdim, m.scale, **kw))
+                pairs = sum(min(t + 1, win) for t in range(rows))
+                put(key, ms, flops=2 * pairs * m.heads * (m.dim + m.vdim))
+            else:
+                splits = max(1, min(16, (4 * eng._sms) // (rows * m.heads), (win + 31) // 32))
+                ms = timeit(lambda: ops.attn_ragged(qbuf, kc, vc, proj, mix, row_ent, ent, eng.kv.page_table, m.heads, m.kv_heads,
+                                                    m.dim, m.vdim, m.scale, splits=splits, part=eng._apart_att if splits > 1 else None, **kw))
+                put(key, ms, byt=min(start + 1, win) * m.kv_heads * (m.dim + m.vdim) * eb)
+        # feed-forward: the gelu epilogue, the experts
+        li_d = next(i for i, L in enumerate(spec.layers) if L.ff)
+        L, Pd = spec.layers[li_d], eng.layers[li_d]
+        act = torch.empty(rows, L.ff, dtype=E, device=dev)
+        ms = timeit(lambda: ops.linear_gated_act(he, Pd["w_gu"], Pd["ff_act"], None, out=act), n=3, reps=3)
+        ms2 = timeit(lambda: ops.linear_gated_silu(he, Pd["w_gu"], out=act), n=3, reps=3)
+        for key, t in ((f"{tag}_ff_gate_up_gelu", ms), (f"{tag}_ff_gate_up_silu", ms2)):
+            put(key, t, flops=4 * rows * W * L.ff) if rows > 1 else put(key, t, byt=2 * W * L.ff * eb)
+        gu = torch.empty(rows, P["w_gu"].shape[0], dtype=E, device=dev)
+        act = torch.empty(rows, e.total_ff, dtype=E, device=dev)
+        y2 = torch.empty(rows, W, dtype=E, device=dev)
+        ms_gu = timeit(lambda: eng._lin(he, P["w_gu"], gu), n=3, reps=3)
+        ms_act = timeit(lambda: ops.moe_act(gu, route["wts"], act, e.experts, e.ff, 0.0, silu=True))
+        ms_dn = timeit(lambda: eng._lin(act, P["w_down"], y2), n=3, reps=3)
+        put(f"{tag}_moe_act", ms_act, byt=rows * (e.total_ff + 2 * e.top * e.ff) * eb)
+        if rows > 1:
+            put(f"{tag}_moe_projections", ms_gu + ms_dn, flops=2 * rows * 3 * W * e.top * e.ff)
+            res[f"{tag}_moe_projections"]["of_bf16_peak_all_experts"] = round(2 * rows * 3 * W * e.total_ff / ((ms_gu + ms_dn) / 1e3) / tc, 4)
+        else:
+            put(f"{tag}_moe_projections_all_experts", ms_gu + ms_dn, byt=3 * W * e.total_ff * eb)
+            act_sel = torch.empty(rows, e.top * e.ff, dtype=E, device=dev)
+            ms = timeit(lambda: ops.moe_sel(he, P["w_gu"], P["w_down"], route["sel_idx"], route["sel_w"], act_sel, y2, e.experts, e.top,
+                                            e.ff, 0.0, silu=True))
+            put(f"{tag}_moe_chosen_experts", ms, byt=3 * W * e.top * e.ff * eb)
+    eng.close_sequence(slot)
+    return res
+
 
 def hybrid_kernel_times(eng, spec, T, peaks):
     """Each kernel of the ragged path alone at the step sizes of the comparison: a T-token portion (prefill) and one
@@ -1217,6 +1401,8 @@ def main():
                     help="instead of the default workload: the Fubepel design beside the Sokevik design at equal sizes")
     ap.add_argument("--compare-gimudra", action="store_true",
                     help="prefill / decode throughput of the Gimudra design beside the Togalorn and Sokevik designs at equal sizes")
+    ap.add_argument("--compare-salizen", action="store_true",
+                    help="prefill / decode throughput of the Salizen design beside the Togalorn and Gimudra designs at equal sizes")
     ap.add_argument("--hybrid-sizes", default="1b,8b")
     args = ap.parse_args()
 
@@ -1247,6 +1433,10 @@ def main():
     if args.compare_gimudra:
         if rank == 0:
             print(json.dumps(run_gimudra_compare(args, peaks)), flush=True)
+        return
+    if args.compare_salizen:
+        if rank == 0:
+            print(json.dumps(run_salizen_compare(args, peaks)), flush=True)
         return
     if world > 1 or args.gpus > 1:
         from dli_b200.pipeline import run_pipeline_bench
