@@ -115,6 +115,7 @@ SIGNATURES = {
     "dli_head_rmsnorm_gate": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _i, _i, _i, _i, _vp]),
     "dli_streams_close": (_i, [_vp, _vp, _sz, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp, _vp, _vp, _vp, _vp, _vp,
                                _vp, _i, _i, _i, _i, _i, _f, _i, _vp]),
+    "dli_linattn_tc_supported": (_i, [_i, _i, _i, _i, _i, _i]),
     "dli_linattn_scratch_floats": (_sz, [_i, _i, _i, _i]),
     "dli_linattn_ragged": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _vp, _i, _vp, _i, _i,
                                 _vp, _vp, _f, _i, _vp, _vp, _i, _vp, _i, _vp]),

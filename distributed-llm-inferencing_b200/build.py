@@ -39,6 +39,7 @@ SOURCES = [
     "prenorm_rows.cu",
     "stream_rows.cu",
     "linear_attn.cu",
+    "linear_attn_tc.cu",
 ]
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]

@@ -194,7 +194,8 @@ __device__ __forceinline__ float gelu_new_f(float x) {
 __device__ __forceinline__ float gated_combine(float gte, float up, const float* __restrict__ act) {
   if (act == nullptr) return round_bf16(silu_f(gte)) * up;
   const float lim = act[0], alpha = act[1];
-  if (lim <= 0.f) return gelu_new_f(gte) * up;
+  // 0.5 (1 + tanh z) = 1 / (1 + e^(-2z)): the tanh form of gelu at silu's cost
+  if (lim <= 0.f) return gte / (1.0f + expf(-1.5957691216057308f * (gte + 0.044715f * gte * gte * gte))) * up;
   const float g = fminf(gte, lim), u = fminf(fmaxf(up, -lim), lim);
   return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
 }

@@ -13,47 +13,15 @@
 //                     o_t   = S_in^T (e^(c_t) q_t) + sum_(s<=t) (sum_d q_t[d] k_s[d] e^(c_t[d] - c_s[d])) v_s
 //                     S_out = diag(e^(c_L)) S_in + sum_s (e^(c_L - c_s) k_s) v_s^T
 //                   Every exponent is <= 0.
-//   blocks of 64 rows in parallel (tiles): what a block adds to the state, an elementwise carry in order, read-outs.
+//   tiles of 64 rows in parallel: what a tile adds to the state, an elementwise carry in order, read-outs; bf16 engines run
+//                   the first and the last on the tensor cores (linear_attn_tc.cu)
 #include <math.h>
 
-#include "common.cuh"
+#include "linear_attn.cuh"
 
 namespace dli {
 
-template <typename E> __device__ __forceinline__ float l_to_f(E v);
-template <> __device__ __forceinline__ float l_to_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ float l_to_f<bf16>(bf16 v) { return __bfloat162float(v); }
-
-struct LinAttn {
-  const int32_t* ent;
-  int H, D, V;
-  int ldp, q_off, k_off, v_off;
-  int silu;                 // SiLU on q, k and v
-  float q_scale, k_scale;
-  const float* cos_t;       // [positions, rd/2]
-  const float* sin_t;
-  int rd;
-  const float* log_decay;   // [H]: log of the fixed decay, or NULL:
-  int a_off, rank;          // columns of a_t
-  const float* a2;          // [H*D, rank]
-  const float* a2_b;        // [H*D]
-  float inv_tau;
-};
-
-// one prepared entry of q or k: column `base + i` of the projection row, i within the head
-template <typename E>
-__device__ __forceinline__ float la_qk(const E* pr, int base, int i, const LinAttn& a, int pos, float scale) {
-  float u = l_to_f(pr[base + i]);
-  if (a.silu) u = silu_f(u);
-  if (i < a.rd) {
-    const int half = a.rd >> 1, j = i < half ? i : i - half;
-    float p = l_to_f(pr[base + (i < half ? i + half : j)]);
-    if (a.silu) p = silu_f(p);
-    const float c = a.cos_t[(size_t)pos * half + j], s = a.sin_t[(size_t)pos * half + j];
-    u = i < half ? u * c - p * s : u * c + p * s;
-  }
-  return u * scale;
-}
+__device__ __forceinline__ float la_log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
 // log w_t of key channel `ch` (head-major): (1/tau) log sigmoid(A2[ch] . a_t + b[ch])
 template <typename E>
@@ -61,8 +29,7 @@ __device__ __forceinline__ float la_log_decay(const E* pr, int ch, const LinAttn
   const float* w = a.a2 + (size_t)ch * a.rank;
   float z = 0.f;
   for (int r = 0; r < a.rank; ++r) z = fmaf(w[r], l_to_f(pr[a.a_off + r]), z);
-  z += a.a2_b[ch];
-  return (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * a.inv_tau;
+  return la_log_sigmoid(z + a.a2_b[ch]) * a.inv_tau;
 }
 
 // ---- row by row ---------------------------------------------------------------------------------------------------
@@ -161,19 +128,45 @@ linattn_rows_kernel(const E* __restrict__ proj, float* __restrict__ S, float* __
 }
 
 // ---- log decays of every row (portions): lg [rows, H*D] -----------------------------------------------------------------
+// 16 rows x 256 channels per CTA: a thread holds 16 entries of its channel's row of A2 at a time, the rows' a_t are in shared
+// memory.
+constexpr int kLdRows = 16;
 template <typename E>
 __global__ void __launch_bounds__(256)
-linattn_log_decay_kernel(const E* __restrict__ proj, float* __restrict__ lg, LinAttn a) {
+linattn_log_decay_kernel(const E* __restrict__ proj, float* __restrict__ lg, LinAttn a, int rows) {
+  __shared__ __align__(16) float as[kLdRows][16];
   pdl_wait();
   pdl_trigger();
-  const size_t row = blockIdx.x;
-  const int n = a.H * a.D;
-  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < n; c += blockDim.x * gridDim.y)
-    lg[row * n + c] = la_log_decay(proj + row * a.ldp, c, a);
+  const int n = a.H * a.D, row0 = blockIdx.x * kLdRows, ch = blockIdx.y * 256 + threadIdx.x;
+  float z[kLdRows];
+  const float b = ch < n ? a.a2_b[ch] : 0.f;
+#pragma unroll
+  for (int t = 0; t < kLdRows; ++t) z[t] = 0.f;
+  for (int r0 = 0; r0 < a.rank; r0 += 16) {
+    __syncthreads();
+    {
+      const int t = threadIdx.x >> 4, r = r0 + (threadIdx.x & 15);
+      as[t][threadIdx.x & 15] = (row0 + t < rows && r < a.rank) ? l_to_f(proj[(size_t)(row0 + t) * a.ldp + a.a_off + r]) : 0.f;
+    }
+    float w[16];
+#pragma unroll
+    for (int r = 0; r < 16; ++r) w[r] = (ch < n && r0 + r < a.rank) ? a.a2[(size_t)ch * a.rank + r0 + r] : 0.f;
+    __syncthreads();
+#pragma unroll
+    for (int t = 0; t < kLdRows; ++t)
+#pragma unroll
+      for (int r = 0; r < 16; r += 4) {
+        const float4 f = *reinterpret_cast<const float4*>(&as[t][r]);
+        z[t] = fmaf(w[r], f.x, z[t]); z[t] = fmaf(w[r + 1], f.y, z[t]); z[t] = fmaf(w[r + 2], f.z, z[t]); z[t] = fmaf(w[r + 3], f.w, z[t]);
+      }
+  }
+  if (ch >= n) return;
+#pragma unroll
+  for (int t = 0; t < kLdRows; ++t)
+    if (row0 + t < rows) lg[(size_t)(row0 + t) * n + ch] = la_log_sigmoid(z[t] + b) * a.inv_tau;
 }
 
 // ---- blocks -------------------------------------------------------------------------------------------------------------
-constexpr int kLaTile = 64;   // rows per tile of the parallel form
 constexpr int kLaL = 16;      // rows per block
 constexpr int kLaP = 20;      // padded row of the transposed blocks
 constexpr int kLaVc = 64;     // value columns per CTA
@@ -414,9 +407,16 @@ static int launch_blocks(const void* proj, const float* lg, float* S, float* o, 
     LA_BLOCKS(0, n_ent, "linattn_blocks");
     return DLI_OK;
   }
-  LA_BLOCKS(1, n_tiles, "linattn_local");
+  const bool tc = sizeof(E) == 2 && linattn_tc_supported(a);
+  if (tc) {
+    const int rc = linattn_tc_local(proj, lg, a, tiles, n_tiles, scr_u, scr_w, s);
+    if (rc != DLI_OK) return rc;
+  } else {
+    LA_BLOCKS(1, n_tiles, "linattn_local");
+  }
   DLI_LAUNCH("linattn_carry", linattn_carry_kernel, dim3(n_ent, a.H, (a.D * a.V + 255) / 256), dim3(256), 0, s, a.ent, tiles, n_tiles,
              S, scr_u, (const float*)scr_w, a.H, a.D, a.V);
+  if (tc) return linattn_tc_out(proj, lg, o, a, tiles, n_tiles, scr_u, s);
   LA_BLOCKS(3, n_tiles, "linattn_out");
 #undef LA_BLOCKS
   return DLI_OK;
@@ -427,6 +427,14 @@ static int launch_blocks(const void* proj, const float* lg, float* S, float* o, 
 using namespace dli;
 
 extern "C" {
+
+int dli_linattn_tc_supported(int D, int V, int gated, int silu, int rd, int dt) {
+  LinAttn a{};
+  a.D = D; a.V = V; a.silu = silu; a.rd = rd;
+  static const float one = 0.f;
+  a.log_decay = gated ? nullptr : &one;
+  return dt == 0 && linattn_tc_supported(a) ? 1 : 0;
+}
 
 size_t dli_linattn_scratch_floats(int n_tiles, int H, int D, int V) {
   return (size_t)n_tiles * H * D * ((size_t)V + 1);
@@ -455,11 +463,11 @@ int dli_linattn_ragged(const void* proj, float* S, float* o, const int32_t* ent,
     return dt == 0 ? launch_rows<bf16>(proj, S, o, n_ent, a, s) : launch_rows<float>(proj, S, o, n_ent, a, s);
   if (gated) {
     DLI_CHECK_ARG(lg, "dli_linattn_ragged: portions with a decay per channel need scratch for the log decays");
-    const dim3 grid(rows, (H * D + 1023) / 1024);
-    if (dt == 0) DLI_LAUNCH("linattn_log_decay", linattn_log_decay_kernel<bf16>, grid, dim3(256), 0, s, (const bf16*)proj, lg, a);
-    else DLI_LAUNCH("linattn_log_decay", linattn_log_decay_kernel<float>, grid, dim3(256), 0, s, (const float*)proj, lg, a);
+    const dim3 grid((rows + kLdRows - 1) / kLdRows, (H * D + 255) / 256);
+    if (dt == 0) DLI_LAUNCH("linattn_log_decay", linattn_log_decay_kernel<bf16>, grid, dim3(256), 0, s, (const bf16*)proj, lg, a, rows);
+    else DLI_LAUNCH("linattn_log_decay", linattn_log_decay_kernel<float>, grid, dim3(256), 0, s, (const float*)proj, lg, a, rows);
   }
-  float* scr = (tiles && n_tiles > n_ent) ? scratch : nullptr;  // some entry spans several tiles: all tiles in parallel
+  float* scr = tiles && n_tiles > 0 ? scratch : nullptr;  // with scratch: all tiles in parallel
   if (dt == 0) return gated ? launch_blocks<bf16, true>(proj, lg, S, o, a, n_ent, tiles, n_tiles, scr, s)
                             : launch_blocks<bf16, false>(proj, lg, S, o, a, n_ent, tiles, n_tiles, scr, s);
   return gated ? launch_blocks<float, true>(proj, lg, S, o, a, n_ent, tiles, n_tiles, scr, s)

@@ -946,6 +946,10 @@ def streams_close(x, rows, y=None, mix=None, outw=None, in_next=None, w_next=Non
     return x
 
 
+def linattn_tc_supported(D, V, gated, silu, rd, dtype) -> bool:
+    return dtype == torch.bfloat16 and bool(_lib.load().dli_linattn_tc_supported(int(D), int(V), int(bool(gated)), int(bool(silu)), int(rd), 0))
+
+
 def linattn_scratch_floats(n_tiles, H, D, V) -> int:
     return int(_lib.load().dli_linattn_scratch_floats(int(n_tiles), int(H), int(D), int(V)))
 
@@ -957,12 +961,12 @@ def linattn_ragged(proj, S, o, ent, H, D, V, q_off, k_off, v_off, silu=False, q_
     float32 [rows, H*V].  log_decay float32 [H]: fixed decay per head; else a decay per key channel from columns a_off.. of
     proj through a2 [H*D, rank], a2_b [H*D] (float32) and inv_tau.  blocked: small matrix products (steps with portions of
     prompts; lg float32 scratch [rows, H*D] for a decay per channel), with tiles and scratch of linattn_scratch_floats(...)
-    floats the 64-row tiles of an entry in parallel."""
+    floats all 64-row tiles in parallel (on the tensor cores where linattn_tc_supported)."""
     _req(proj, proj.dtype), _f32(S, o, cos_t, sin_t, log_decay, a2, a2_b, lg, scratch), _i32(ent, tiles)
     rows, n_ent = proj.shape[0], ent.numel() // 4
     n_tiles = tiles.numel() // 2 if tiles is not None else 0
     gated = log_decay is None
-    par = bool(blocked) and scratch is not None and n_tiles > n_ent
+    par = bool(blocked) and scratch is not None and n_tiles > 0
     if par and scratch.numel() < linattn_scratch_floats(n_tiles, H, D, V):
         raise ValueError("linattn_ragged: scratch too small")
     if o.numel() < rows * H * V or (gated and blocked and lg.numel() < rows * H * D):

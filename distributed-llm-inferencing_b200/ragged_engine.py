@@ -1129,9 +1129,10 @@ class RaggedEngine:
         o = self._oscr[:rows * H * V].view(rows, H * V)
         cos_t, sin_t = self._table(m.rot_base, m.rot_dims, m.rot_scaling) if m.rot_dims else (None, None)
         scr, n_tiles, n_ent = None, d_tiles.numel() // 2, d_ent.numel() // 4
-        if long_step and n_tiles > n_ent and n_ent * H * ((V + 63) // 64) < 4 * self._sms:
-            # some entry spans several 64-row tiles and the (entry, head, 64 value columns) do not fill the GPU: all tiles at
-            # once (bounded scratch, else tiles in order)
+        tc = ops.linattn_tc_supported(D, V, bool(m.tau), m.qkv_silu, m.rot_dims, self.dtype)
+        if long_step and (tc or (n_tiles > n_ent and n_ent * H * ((V + 63) // 64) < 4 * self._sms)):
+            # all 64-row tiles at once: on the tensor cores, or because some entry spans several tiles and the (entry, head, 64
+            # value columns) would not fill the GPU (bounded scratch, else tiles in order)
             need = ops.linattn_scratch_floats(n_tiles, H, D, V)
             if need <= self.mlstm_parallel_max_floats:
                 if getattr(self, "_la_scr", None) is None or self._la_scr.numel() < need:

@@ -21,7 +21,7 @@ down}, l<i>.mlp.router, l<i>.mlp.router.b.
 """
 from __future__ import annotations
 
-from typing import Dict, List, Optional
+from typing import Dict, List
 
 import torch
 
@@ -137,12 +137,11 @@ def model_tensors(spec: HybridSpec, sd: Dict[str, torch.Tensor]) -> dict:
     return out
 
 
-def random_state_dict(spec: HybridSpec, seed: int = 0, std: float = 0.05, device="cpu", rank: Optional[int] = None) -> Dict[str, torch.Tensor]:
+def random_state_dict(spec: HybridSpec, seed: int = 0, std: float = 0.05, device="cpu", rank: int = 16) -> Dict[str, torch.Tensor]:
     """Synthetic weights under the checkpoint's names (benchmarks and tests; there are no checkpoints offline).  rank: size
-    of the decay projection (default: the width / 16)."""
+    of the decay projection."""
     g = torch.Generator(device="cpu").manual_seed(seed)
     W, S = spec.width, spec.streams
-    rank = rank or max(4, W // 16)
 
     def n(*shape, s=std, mean=0.0):
         return (mean + s * torch.randn(tuple(shape), generator=g)).to(torch.bfloat16).to(device)

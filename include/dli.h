@@ -661,7 +661,9 @@ int dli_streams_close(const void* y, float* x, size_t xs_stride, int n_streams, 
  * exp(log_decay[h]), or, with log_decay NULL, per key channel sigmoid(a2 . proj[row, a_off : +rank] + a2_b)^inv_tau
  * (a2 [H*D, rank], a2_b [H*D] fp32).  blocked != 0 (steps with portions of prompts): 16 rows at a time as small matrix
  * products, else row by row; lg: scratch [rows, H*D] for the blocked form with a decay per channel; with tiles (as for
- * dli_attn_ragged_tc) and scratch of dli_linattn_scratch_floats floats the 64-row tiles of an entry run in parallel. */
+ * dli_attn_ragged_tc) and scratch of dli_linattn_scratch_floats floats the 64-row tiles of all entries run in parallel, on
+ * the tensor cores where dli_linattn_tc_supported (bf16 rows; operands that are not exact in bf16 as the sum of two). */
+int dli_linattn_tc_supported(int D, int V, int gated, int silu, int rd, int dt);
 size_t dli_linattn_scratch_floats(int n_tiles, int H, int D, int V);
 int dli_linattn_ragged(const void* proj, float* S, float* o, const int32_t* ent, int n_ent, int rows, int H, int D, int V, int ldp,
                        int q_off, int k_off, int v_off, int silu, float q_scale, float k_scale, const float* cos_t,
