@@ -389,7 +389,7 @@ static int launch_rows(const void* proj, float* S, float* o, int n_ent, const Li
 }
 
 template <typename E, bool gated>
-static int launch_blocks(const void* proj, const float* lg, float* S, float* o, const LinAttn& a, int n_ent, const int32_t* tiles,
+static int launch_blocks(const void* proj, float* lg, float* S, float* o, const LinAttn& a, int n_ent, int rows, const int32_t* tiles,
                          int n_tiles, float* scratch, cudaStream_t s) {
   const size_t smem = linattn_block_smem(a.D, gated);
   const int nz = (a.V + kLaVc - 1) / kLaVc;
@@ -407,16 +407,16 @@ static int launch_blocks(const void* proj, const float* lg, float* S, float* o, 
     LA_BLOCKS(0, n_ent, "linattn_blocks");
     return DLI_OK;
   }
-  const bool tc = sizeof(E) == 2 && linattn_tc_supported(a);
+  const bool tc = sizeof(E) == 2 && lg && linattn_tc_supported(a);
   if (tc) {
-    const int rc = linattn_tc_local(proj, lg, a, tiles, n_tiles, scr_u, scr_w, s);
+    const int rc = linattn_tc_local(proj, lg, a, rows, tiles, n_tiles, scr_u, scr_w, s);
     if (rc != DLI_OK) return rc;
   } else {
     LA_BLOCKS(1, n_tiles, "linattn_local");
   }
   DLI_LAUNCH("linattn_carry", linattn_carry_kernel, dim3(n_ent, a.H, (a.D * a.V + 255) / 256), dim3(256), 0, s, a.ent, tiles, n_tiles,
              S, scr_u, (const float*)scr_w, a.H, a.D, a.V);
-  if (tc) return linattn_tc_out(proj, lg, o, a, tiles, n_tiles, scr_u, s);
+  if (tc) return linattn_tc_out(proj, lg, o, a, rows, tiles, n_tiles, scr_u, s);
   LA_BLOCKS(3, n_tiles, "linattn_out");
 #undef LA_BLOCKS
   return DLI_OK;
@@ -468,10 +468,10 @@ int dli_linattn_ragged(const void* proj, float* S, float* o, const int32_t* ent,
     else DLI_LAUNCH("linattn_log_decay", linattn_log_decay_kernel<float>, grid, dim3(256), 0, s, (const float*)proj, lg, a, rows);
   }
   float* scr = tiles && n_tiles > 0 ? scratch : nullptr;  // with scratch: all tiles in parallel
-  if (dt == 0) return gated ? launch_blocks<bf16, true>(proj, lg, S, o, a, n_ent, tiles, n_tiles, scr, s)
-                            : launch_blocks<bf16, false>(proj, lg, S, o, a, n_ent, tiles, n_tiles, scr, s);
-  return gated ? launch_blocks<float, true>(proj, lg, S, o, a, n_ent, tiles, n_tiles, scr, s)
-               : launch_blocks<float, false>(proj, lg, S, o, a, n_ent, tiles, n_tiles, scr, s);
+  if (dt == 0) return gated ? launch_blocks<bf16, true>(proj, lg, S, o, a, n_ent, rows, tiles, n_tiles, scr, s)
+                            : launch_blocks<bf16, false>(proj, lg, S, o, a, n_ent, rows, tiles, n_tiles, scr, s);
+  return gated ? launch_blocks<float, true>(proj, lg, S, o, a, n_ent, rows, tiles, n_tiles, scr, s)
+               : launch_blocks<float, false>(proj, lg, S, o, a, n_ent, rows, tiles, n_tiles, scr, s);
 }
 
 }  // extern "C"

@@ -41,11 +41,12 @@ __device__ __forceinline__ float la_qk(const E* pr, int base, int i, const LinAt
 
 constexpr int kLaTile = 64;   // rows per tile of the tile-parallel forms
 
-// linear_attn_tc.cu: the tiles' state contributions and read-outs on the tensor cores (bf16 projection rows)
+// linear_attn_tc.cu: the tiles' state contributions and read-outs on the tensor cores (bf16 projection rows).  row_scr: the
+// rows' log decays [rows, H*D], or, with a fixed decay, scratch of rows * (2HD + HV) floats that local fills and out reads.
 bool linattn_tc_supported(const LinAttn& a);
-int linattn_tc_local(const void* proj, const float* lg, const LinAttn& a, const int32_t* tiles, int n_tiles, float* scr_u,
+int linattn_tc_local(const void* proj, float* row_scr, const LinAttn& a, int rows, const int32_t* tiles, int n_tiles, float* scr_u,
                      float* scr_w, cudaStream_t s);
-int linattn_tc_out(const void* proj, const float* lg, float* o, const LinAttn& a, const int32_t* tiles, int n_tiles,
+int linattn_tc_out(const void* proj, float* row_scr, float* o, const LinAttn& a, int rows, const int32_t* tiles, int n_tiles,
                    const float* scr_u, cudaStream_t s);
 
 }  // namespace dli

@@ -14,6 +14,10 @@
 // k_s e^(r - c_s) of the earlier rows have exponents <= 0.  Inside the block r - c_s >= 0 is the block's own decay: below
 // kSafeLog2 it is multiplied in all the same (bf16 has fp32's exponent range), above it the block's 16 x 16 scores are
 // summed directly with e^(c_t - c_s) per channel.
+//
+// The key dimension goes through shared memory 64 channels at a time, so that several CTAs share an SM and one's loads
+// overlap another's products.  With a fixed decay, q, k and v are prepared once per row by linattn_prep_kernel (SiLU,
+// rotation, factors) and split into hi and lo rows there.
 #include <math.h>
 
 #include "linear_attn.cuh"
@@ -27,17 +31,15 @@ constexpr int kTcVp = kTcVc + 8;    // padded row (an odd number of 16-byte piec
 constexpr float kSafeLog2 = 58.f;
 constexpr float kLog2e = 1.4426950408889634f;
 
-static inline size_t tc_local_smem(int D, bool gated) {
-  return 2 * ((size_t)2 * kLaTile * (D + 8) + (size_t)(gated ? 1 : 2) * kLaTile * kTcVp);
-}
-static inline size_t tc_out_smem(int D, bool gated) {
-  return 2 * ((size_t)(gated ? 2 : 4) * kLaTile * (D + 8) + (size_t)(gated ? 1 : 2) * kLaTile * kTcVp + (size_t)2 * D * kTcVp) +
-         (gated ? 4 * (size_t)kLaTile * (D + 8) : 0);
-}
+constexpr int kTcDc = 64;           // key channels per pass
+constexpr int kTcDp = kTcDc + 8;
+constexpr int kTcRows = kLaTile * kTcDp;  // elements of one [64][72] block
+
+static inline size_t tc_local_smem(bool gated) { return 2 * (size_t)kTcRows * (gated ? 3 : 4); }
+static inline size_t tc_out_smem(bool gated) { return gated ? 2 * (size_t)kTcRows * 5 + 4 * (size_t)kTcRows : 2 * (size_t)kTcRows * 8; }
 
 bool linattn_tc_supported(const LinAttn& a) {
-  const bool gated = a.log_decay == nullptr;
-  return a.D % 16 == 0 && a.V % 8 == 0 && tc_out_smem(a.D, gated) <= 220 * 1024 && !(gated && (a.silu || a.rd));
+  return a.D % 16 == 0 && a.V % 8 == 0 && !(a.log_decay == nullptr && (a.silu || a.rd));
 }
 
 __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
@@ -51,156 +53,207 @@ struct TcTile {
   int pos0, nb;     // its position, rows in the tile
 };
 
-// The prepared q or k (columns `base` ..) of the tile's rows as hi + lo (both [64][D+8]); rows past the tile: zeros.
-// wexp: log2 of a factor per row step, applied as 2^(wexp * (nb - 1 - t)) (0: none).
-__device__ __forceinline__ void stage_rows(const bf16* __restrict__ proj, int base, const LinAttn& a, const TcTile& tl, float scale,
-                                           float wexp, bf16* __restrict__ hi, bf16* __restrict__ lo) {
-  const int D = a.D, DP = D + 8, half = a.rd >> 1, np = D >> 1;
-  for (int i = threadIdx.x; i < kLaTile * np; i += kTcThreads) {
-    const int t = i / np, p = i - t * np;
-    // a rotated pair (p, p + half), or two neighbours behind the rotated dimensions
-    const bool hp = p < half;
-    const int i0 = hp ? p : 2 * p, i1 = hp ? p + half : 2 * p + 1;
-    float u = 0.f, v = 0.f;
-    if (t < tl.nb) {
-      const bf16* pr = proj + (tl.row0 + t) * a.ldp + base;
-      u = __bfloat162float(pr[i0]);
-      v = __bfloat162float(pr[i1]);
-      if (a.silu) { u = silu_f(u); v = silu_f(v); }
-      if (hp) {
-        const size_t at = (size_t)(tl.pos0 + t) * half + p;
-        const float c = a.cos_t[at], s = a.sin_t[at], u2 = u * c - v * s;
-        v = v * c + u * s;
-        u = u2;
+// ---- fixed decay: q | k | v of every row, prepared, as a row of hi and a row of lo parts [2HD + HV] each ----------------
+// An item is W consecutive dimensions of a head, with the W partners half a rotation away where they are rotated.
+struct LinPrep {
+  const int32_t* ent;
+  const int32_t* tiles;
+  bf16* hi;
+  bf16* lo;
+};
+
+template <int W>
+__global__ void __launch_bounds__(256)
+linattn_prep_kernel(const bf16* __restrict__ proj, LinAttn a, LinPrep p) {
+  pdl_wait();
+  pdl_trigger();
+  // one CTA per (tile, 8 of its rows)
+  const int4 e = reinterpret_cast<const int4*>(p.ent)[p.tiles[2 * blockIdx.x]];  // slot, first row, rows, first position
+  const int b0 = p.tiles[2 * blockIdx.x + 1] + 8 * blockIdx.y;
+  const int nb = min(8, e.z - b0);
+  const int half = a.rd >> 1, nrot = half / W, nqk = nrot + (a.D - a.rd) / W, nv = a.V / W;
+  const int per_row = a.H * (2 * nqk + nv), C = a.H * (2 * a.D + a.V);
+  for (int i = threadIdx.x; i < nb * per_row; i += 256) {
+    const int t = i / per_row;
+    int it = i - t * per_row;
+    const size_t row = (size_t)(e.y + b0 + t);
+    // which of q, k, v; head; item within the head
+    const int part = it < a.H * nqk ? 0 : (it < 2 * a.H * nqk ? 1 : 2);
+    it -= part == 0 ? 0 : (part == 1 ? a.H * nqk : 2 * a.H * nqk);
+    const int n = part == 2 ? nv : nqk, sz = part == 2 ? a.V : a.D;
+    const int h = it / n, x = it - h * n;
+    const bool rot = part < 2 && x < nrot;
+    const int d0 = part == 2 ? x * W : (rot ? x * W : a.rd + (x - nrot) * W);
+    const int off = part == 0 ? a.q_off : (part == 1 ? a.k_off : a.v_off);
+    const bf16* src = proj + row * a.ldp + off + h * sz + d0;
+    const size_t dst = row * C + (part == 0 ? 0 : (part == 1 ? a.H * a.D : 2 * a.H * a.D)) + h * sz + d0;
+    const float f = part == 0 ? a.q_scale : (part == 1 ? a.k_scale : 1.f);
+    float u[W], v[W];
+    auto load = [&](const bf16* s, float (&r)[W]) {
+      if constexpr (W == 8) unpack8(ld_16B(s), r);
+      else r[0] = __bfloat162float(*s);
+      if (a.silu) {
+#pragma unroll
+        for (int k = 0; k < W; ++k) r[k] = silu_f(r[k]);
       }
-      const float f = wexp != 0.f ? scale * exp2f(wexp * (float)(tl.nb - 1 - t)) : scale;
-      u *= f;
-      v *= f;
-    }
-    uint32_t h, l;
-    split2(u, v, h, l);
-    bf16* hr = hi + t * DP;
-    bf16* lr = lo + t * DP;
-    if (hp) {
-      hr[i0] = __ushort_as_bfloat16((unsigned short)(h & 0xffffu)); hr[i1] = __ushort_as_bfloat16((unsigned short)(h >> 16));
-      lr[i0] = __ushort_as_bfloat16((unsigned short)(l & 0xffffu)); lr[i1] = __ushort_as_bfloat16((unsigned short)(l >> 16));
+    };
+    auto store = [&](size_t at, const float (&r)[W]) {
+      float l[W];
+#pragma unroll
+      for (int k = 0; k < W; ++k) l[k] = r[k] - round_bf16(r[k]);
+      if constexpr (W == 8) {
+        st_16B(p.hi + at, pack8(r));
+        st_16B(p.lo + at, pack8(l));
+      } else {
+        p.hi[at] = __float2bfloat16_rn(r[0]);
+        p.lo[at] = __float2bfloat16_rn(l[0]);
+      }
+    };
+    load(src, u);
+    if (rot) {
+      load(src + half, v);
+      const size_t tb = (size_t)(e.w + b0 + t) * half + d0;
+#pragma unroll
+      for (int k = 0; k < W; ++k) {
+        const float c = a.cos_t[tb + k], s = a.sin_t[tb + k];
+        const float u2 = (u[k] * c - v[k] * s) * f;
+        v[k] = (v[k] * c + u[k] * s) * f;
+        u[k] = u2;
+      }
+      store(dst, u);
+      store(dst + half, v);
     } else {
-      *reinterpret_cast<uint32_t*>(hr + i0) = h;
-      *reinterpret_cast<uint32_t*>(lr + i0) = l;
+#pragma unroll
+      for (int k = 0; k < W; ++k) u[k] *= f;
+      store(dst, u);
     }
   }
 }
 
-// The rows' raw bf16 columns [64][n] (n a multiple of 8) into rows of `ld` elements, zeros past the tile and past n_valid.
-__device__ __forceinline__ void stage_raw(const bf16* __restrict__ proj, int base, const LinAttn& a, const TcTile& tl, int n, int n_valid,
-                                          bf16* __restrict__ dst, int ld) {
-  const bool al = (a.ldp % 8 == 0) && (base % 8 == 0) && (reinterpret_cast<uintptr_t>(proj) & 15u) == 0;
-  const int nc = n >> 3;
-  for (int i = threadIdx.x; i < kLaTile * nc; i += kTcThreads) {
-    const int t = i / nc, c = (i - t * nc) * 8;
-    uint4 u = make_uint4(0, 0, 0, 0);
-    if (t < tl.nb && c < n_valid) {
-      const bf16* src = proj + (tl.row0 + t) * a.ldp + base + c;
-      if (al) {
-        u = ld_16B(src);
-      } else {
-        const unsigned short* us = reinterpret_cast<const unsigned short*>(src);
+// 64 columns of the tile's rows (row stride ld, the first n_valid exist) into a [64][72] block; zeros elsewhere.  The copies
+// are asynchronous where the rows' alignment allows: cp_async_wait before the barrier.
+__device__ __forceinline__ void stage_raw(const bf16* __restrict__ src, size_t ld, const TcTile& tl, int n_valid, bool al, bf16* __restrict__ dst) {
+  const uint32_t sd = smem_u32(dst);
+#pragma unroll
+  for (int i = threadIdx.x; i < kLaTile * 8; i += kTcThreads) {
+    const int t = i >> 3, c = (i & 7) * 8;
+    const bool ok = t < tl.nb && c < n_valid;
+    const bf16* s = src + (ok ? t * ld + c : 0);
+    if (al) {
+      cp_async_16B(sd + (t * kTcDp + c) * 2, s, ok ? 16 : 0);
+    } else {
+      uint4 u = make_uint4(0, 0, 0, 0);
+      if (ok) {
+        const unsigned short* us = reinterpret_cast<const unsigned short*>(s);
         u.x = us[0] | ((uint32_t)us[1] << 16); u.y = us[2] | ((uint32_t)us[3] << 16);
         u.z = us[4] | ((uint32_t)us[5] << 16); u.w = us[6] | ((uint32_t)us[7] << 16);
       }
+      *reinterpret_cast<uint4*>(dst + t * kTcDp + c) = u;
     }
-    *reinterpret_cast<uint4*>(dst + t * ld + c) = u;
   }
 }
 
-// v of the tile: gated: raw columns; fixed decay: SiLU if asked for, as hi + lo
-template <bool gated>
-__device__ __forceinline__ void stage_values(const bf16* __restrict__ proj, int h, int v0, const LinAttn& a, const TcTile& tl,
-                                             bf16* __restrict__ vh, bf16* __restrict__ vl) {
-  const int base = a.v_off + h * a.V + v0, nv = min(kTcVc, a.V - v0);
-  if constexpr (gated) {
-    stage_raw(proj, base, a, tl, kTcVc, nv, vh, kTcVp);
-  } else {
-    for (int i = threadIdx.x; i < kLaTile * (kTcVc / 2); i += kTcThreads) {
-      const int t = i / (kTcVc / 2), c = 2 * (i % (kTcVc / 2));
-      float x = 0.f, y = 0.f;
-      if (t < tl.nb && c < nv) {
-        const bf16* src = proj + (tl.row0 + t) * a.ldp + base + c;
-        x = __bfloat162float(src[0]);
-        y = __bfloat162float(src[1]);
-        if (a.silu) { x = silu_f(x); y = silu_f(y); }
-      }
-      uint32_t hi, lo;
-      split2(x, y, hi, lo);
-      *reinterpret_cast<uint32_t*>(vh + t * kTcVp + c) = hi;
-      *reinterpret_cast<uint32_t*>(vl + t * kTcVp + c) = lo;
-    }
-  }
+// may 8 consecutive columns from `base` on be copied as 16 bytes?
+__device__ __forceinline__ bool raw_aligned(const bf16* p, size_t ld, int base) {
+  return ld % 8 == 0 && base % 8 == 0 && (reinterpret_cast<uintptr_t>(p) & 15u) == 0;
 }
 
 // ---- what a tile adds to the state: U [D, 64 columns] -------------------------------------------------------------------
+// Fixed decay: the weights w^(L-1-s) go onto the values (all channels share them); decay per channel: onto the keys.
 template <bool gated>
 __global__ void __launch_bounds__(kTcThreads)
-linattn_tc_local_kernel(const bf16* __restrict__ proj, const float* __restrict__ lg, LinAttn a, const int32_t* __restrict__ tiles,
-                        float* __restrict__ scr_u, float* __restrict__ scr_w) {
+linattn_tc_local_kernel(const bf16* __restrict__ proj, const bf16* __restrict__ hi, const bf16* __restrict__ lo,
+                        const float* __restrict__ lg, LinAttn a, const int32_t* __restrict__ tiles, float* __restrict__ scr_u,
+                        float* __restrict__ scr_w) {
   extern __shared__ __align__(16) uint8_t sm_raw[];
-  const int D = a.D, DP = D + 8;
-  bf16* kh = reinterpret_cast<bf16*>(sm_raw);   // [64][D+8] k_s e^(c_L - c_s), hi
-  bf16* kl = kh + kLaTile * DP;                 // lo
-  bf16* vh = kl + kLaTile * DP;                 // [64][72]
-  bf16* vl = vh + kLaTile * kTcVp;              // fixed decay only
+  const int D = a.D;
+  bf16* kh = reinterpret_cast<bf16*>(sm_raw);   // [64][72] keys, hi
+  bf16* kl = kh + kTcRows;                      // lo
+  bf16* vh = kl + kTcRows;                      // [64][72] values
+  bf16* vl = vh + kTcRows;                      // fixed decay only
   pdl_wait();
   pdl_trigger();
   const int4 e = reinterpret_cast<const int4*>(a.ent)[tiles[2 * blockIdx.x]];  // slot, first row, rows, first position
   const int b0 = tiles[2 * blockIdx.x + 1], h = blockIdx.y, v0 = blockIdx.z * kTcVc;
   const TcTile tl{(size_t)(e.y + b0), e.w + b0, min(kLaTile, e.z - b0)};
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int nv = min(kTcVc, a.V - v0), C = a.H * (2 * D + a.V);
   float* wp = scr_w + ((size_t)blockIdx.x * a.H + h) * D;
-  stage_values<gated>(proj, h, v0, a, tl, vh, vl);
+  const float l2 = gated ? 0.f : a.log_decay[h] * kLog2e;
   if constexpr (gated) {
-    // a thread per channel walks the rows from the last to the first: c_L - c_s is the sum of the later rows' log decays
-    for (int d = tid; d < D; d += kTcThreads) {
+    const int base = a.v_off + h * a.V + v0;
+    stage_raw(proj + tl.row0 * a.ldp + base, a.ldp, tl, nv, raw_aligned(proj, a.ldp, base), vh);
+  } else {
+    const size_t at = tl.row0 * C + 2 * a.H * D + h * a.V + v0;
+    for (int i = tid; i < kLaTile * 8; i += kTcThreads) {
+      const int t = i >> 3, c = (i & 7) * 8;
+      float x[8], y[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) x[k] = y[k] = 0.f;
+      if (t < tl.nb && c < nv) {
+        unpack8(ld_16B(hi + at + (size_t)t * C + c), x);
+        unpack8(ld_16B(lo + at + (size_t)t * C + c), y);
+        const float f = ex2_ftz(l2 * (float)(tl.nb - 1 - t));
+#pragma unroll
+        for (int k = 0; k < 8; ++k) { x[k] = (x[k] + y[k]) * f; y[k] = x[k] - round_bf16(x[k]); }
+      }
+      st_16B(vh + t * kTcDp + c, pack8(x));
+      st_16B(vl + t * kTcDp + c, pack8(y));
+    }
+    if (blockIdx.z == 0)
+      for (int d = tid; d < D; d += kTcThreads) wp[d] = exp2f(l2 * (float)tl.nb);
+  }
+  const uint32_t skh = smem_u32(kh), skl = smem_u32(kl), svh = smem_u32(vh), svl = smem_u32(vl);
+  const int mi = lane >> 3, r8 = lane & 7, gq = lane >> 2, t4 = lane & 3;
+  float* Up = scr_u + (((size_t)blockIdx.x * a.H + h) * D) * a.V + v0;
+  for (int d0 = 0; d0 < D; d0 += kTcDc) {
+    const int nd = min(kTcDc, D - d0);
+    if (d0) __syncthreads();  // the previous pass's keys have been used
+    if constexpr (gated) {
+      // two threads per channel (rows 0..31 and 32..63) walk their rows from the last to the first: c_L - c_s is the sum of
+      // the later rows' log decays; the earlier half adds the later half's total
+      const int d = tid & 63, part = tid >> 6;
+      const bool ok = d < nd;
+      const float* lp = lg + tl.row0 * ((size_t)a.H * D) + h * D + d0 + d;
+      const bf16* kp = proj + tl.row0 * a.ldp + a.k_off + h * D + d0 + d;
       float r = 0.f;
-      const float* lp = lg + tl.row0 * ((size_t)a.H * D) + h * D + d;
-      const bf16* kp = proj + tl.row0 * a.ldp + a.k_off + h * D + d;
-      for (int t0 = kLaTile - 8; t0 >= 0; t0 -= 8) {
+      if (part == 0 && ok)
+        for (int t = 32; t < tl.nb; ++t) r += lp[(size_t)t * a.H * D] * kLog2e;
+      for (int t0 = part * 32 + 24; t0 >= part * 32; t0 -= 8) {
         float l8[8], k8[8];
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
           const int t = t0 + u;
-          l8[u] = t < tl.nb ? lp[(size_t)t * a.H * D] * kLog2e : 0.f;
-          k8[u] = t < tl.nb ? __bfloat162float(kp[(size_t)t * a.ldp]) * a.k_scale : 0.f;
+          const bool in = ok && t < tl.nb;
+          l8[u] = in ? lp[(size_t)t * a.H * D] * kLog2e : 0.f;
+          k8[u] = in ? __bfloat162float(kp[(size_t)t * a.ldp]) * a.k_scale : 0.f;
         }
 #pragma unroll
         for (int u = 7; u >= 0; --u) {
           const float x = k8[u] * ex2_ftz(r);
           r += l8[u];
-          const bf16 hi = __float2bfloat16_rn(x);
-          kh[(t0 + u) * DP + d] = hi;
-          kl[(t0 + u) * DP + d] = __float2bfloat16_rn(x - __bfloat162float(hi));
+          const bf16 xh = __float2bfloat16_rn(x);
+          kh[(t0 + u) * kTcDp + d] = xh;
+          kl[(t0 + u) * kTcDp + d] = __float2bfloat16_rn(x - __bfloat162float(xh));
         }
       }
-      if (blockIdx.z == 0) wp[d] = ex2_ftz(r);
+      if (blockIdx.z == 0 && part == 0 && ok) wp[d0 + d] = ex2_ftz(r);
+    } else {
+      const size_t at = tl.row0 * C + a.H * D + h * D + d0;
+      stage_raw(hi + at, C, tl, nd, true, kh);
+      stage_raw(lo + at, C, tl, nd, true, kl);
     }
-  } else {
-    const float l2 = a.log_decay[h] * kLog2e;
-    stage_rows(proj, a.k_off + h * D, a, tl, a.k_scale, l2, kh, kl);
-    if (blockIdx.z == 0)
-      for (int d = tid; d < D; d += kTcThreads) wp[d] = exp2f(l2 * (float)tl.nb);
-  }
-  __syncthreads();
-  const uint32_t skh = smem_u32(kh), skl = smem_u32(kl), svh = smem_u32(vh), svl = smem_u32(vl);
-  const int mi = lane >> 3, r8 = lane & 7, gq = lane >> 2, t4 = lane & 3;
-  const int nv = min(kTcVc, a.V - v0);
-  float* Up = scr_u + (((size_t)blockIdx.x * a.H + h) * D) * a.V + v0;
-  for (int mt = warp; mt < D / 16; mt += 4) {
+    cp_async_commit();
+    cp_async_wait<0>();
+    __syncthreads();
+    if (warp * 16 >= nd) continue;
     float acc[8][4];
 #pragma unroll
     for (int i = 0; i < 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
 #pragma unroll
     for (int ks = 0; ks < 4; ++ks) {
       uint32_t ah[4], al[4];
-      const uint32_t aoff = ((ks * 16 + (mi >> 1) * 8 + r8) * DP + mt * 16 + (mi & 1) * 8) * 2;
+      const uint32_t aoff = ((ks * 16 + (mi >> 1) * 8 + r8) * kTcDp + warp * 16 + (mi & 1) * 8) * 2;
       ldmatrix_x4_trans(ah, skh + aoff);
       ldmatrix_x4_trans(al, skl + aoff);
 #pragma unroll
@@ -225,7 +278,7 @@ linattn_tc_local_kernel(const bf16* __restrict__ proj, const float* __restrict__
       if (c < nv) {
 #pragma unroll
         for (int r = 0; r < 2; ++r)
-          *reinterpret_cast<float2*>(Up + (size_t)(mt * 16 + gq + 8 * r) * a.V + c) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
+          *reinterpret_cast<float2*>(Up + (size_t)(d0 + warp * 16 + gq + 8 * r) * a.V + c) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
       }
     }
   }
@@ -234,74 +287,40 @@ linattn_tc_local_kernel(const bf16* __restrict__ proj, const float* __restrict__
 // ---- read-outs ----------------------------------------------------------------------------------------------------------
 // Warp w owns rows 16 w .. 16 w + 15 of the tile and all 64 columns; its keys are the 16-row blocks 0 .. w.
 template <bool gated>
-__global__ void __launch_bounds__(kTcThreads)
-linattn_tc_out_kernel(const bf16* __restrict__ proj, const float* __restrict__ lg, float* __restrict__ o, LinAttn a,
-                      const int32_t* __restrict__ tiles, const float* __restrict__ scr_u) {
+__global__ void __launch_bounds__(kTcThreads, 3)
+linattn_tc_out_kernel(const bf16* __restrict__ proj, const bf16* __restrict__ hi, const bf16* __restrict__ lo,
+                      const float* __restrict__ lg, float* __restrict__ o, LinAttn a, const int32_t* __restrict__ tiles,
+                      const float* __restrict__ scr_u) {
   extern __shared__ __align__(16) uint8_t sm_raw[];
-  const int D = a.D, DP = D + 8;
-  bf16* qh = reinterpret_cast<bf16*>(sm_raw);        // [64][D+8]
-  bf16* kh = qh + kLaTile * DP;
-  bf16* ql = kh + kLaTile * DP;                      // fixed decay only: the lo parts
-  bf16* kl = gated ? ql : ql + kLaTile * DP;
-  bf16* vh = gated ? ql : kl + kLaTile * DP;         // [64][72]
-  bf16* vl = vh + kLaTile * kTcVp;                   // fixed decay only
-  bf16* sh = gated ? vl : vl + kLaTile * kTcVp;      // [D][72] the incoming state, hi and lo
-  bf16* sl = sh + D * kTcVp;
-  float* C = reinterpret_cast<float*>(sl + D * kTcVp);  // [64][D+8] gated: running log2 decays, inclusive
+  const int D = a.D;
+  bf16* qh = reinterpret_cast<bf16*>(sm_raw);        // [64][72] blocks of 64 channels (values: 64 columns)
+  bf16* kh = qh + kTcRows;
+  bf16* vh = kh + kTcRows;
+  bf16* sh = vh + kTcRows;                           // the incoming state, hi and lo
+  bf16* sl = sh + kTcRows;
+  bf16* ql = sl + kTcRows;                           // fixed decay only: the lo parts
+  bf16* kl = ql + kTcRows;
+  bf16* vl = kl + kTcRows;
+  float* Cs = reinterpret_cast<float*>(sl + kTcRows);  // gated: [64][72] running log2 decays, inclusive
   pdl_wait();
   pdl_trigger();
   const int4 e = reinterpret_cast<const int4*>(a.ent)[tiles[2 * blockIdx.x]];  // slot, first row, rows, first position
   const int b0 = tiles[2 * blockIdx.x + 1], h = blockIdx.y, v0 = blockIdx.z * kTcVc;
   const TcTile tl{(size_t)(e.y + b0), e.w + b0, min(kLaTile, e.z - b0)};
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int nv = min(kTcVc, a.V - v0);
-  stage_values<gated>(proj, h, v0, a, tl, vh, vl);
+  const int nv = min(kTcVc, a.V - v0), C = a.H * (2 * D + a.V);
   if constexpr (gated) {
-    stage_raw(proj, a.q_off + h * D, a, tl, D, D, qh, DP);
-    stage_raw(proj, a.k_off + h * D, a, tl, D, D, kh, DP);
-    for (int d = tid; d < D; d += kTcThreads) {
-      float c = 0.f;
-      const float* lp = lg + tl.row0 * ((size_t)a.H * D) + h * D + d;
-      for (int t0 = 0; t0 < kLaTile; t0 += 8) {
-        float l8[8];
-#pragma unroll
-        for (int u = 0; u < 8; ++u) l8[u] = t0 + u < tl.nb ? lp[(size_t)(t0 + u) * a.H * D] * kLog2e : 0.f;
-#pragma unroll
-        for (int u = 0; u < 8; ++u) { c += l8[u]; C[(t0 + u) * DP + d] = c; }
-      }
-    }
+    const int base = a.v_off + h * a.V + v0;
+    stage_raw(proj + tl.row0 * a.ldp + base, a.ldp, tl, nv, raw_aligned(proj, a.ldp, base), vh);
   } else {
-    stage_rows(proj, a.q_off + h * D, a, tl, a.q_scale, 0.f, qh, ql);
-    stage_rows(proj, a.k_off + h * D, a, tl, a.k_scale, 0.f, kh, kl);
+    const size_t at = tl.row0 * C + 2 * a.H * D + h * a.V + v0;
+    stage_raw(hi + at, C, tl, nv, true, vh);
+    stage_raw(lo + at, C, tl, nv, true, vl);
   }
-  const float* Sp = scr_u + (((size_t)blockIdx.x * a.H + h) * D) * a.V + v0;
-  for (int i = tid; i < D * (kTcVc / 4); i += kTcThreads) {
-    const int d = i / (kTcVc / 4), c = 4 * (i % (kTcVc / 4));
-    float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (c < nv) f = *reinterpret_cast<const float4*>(Sp + (size_t)d * a.V + c);
-    uint2 hi, lo;
-    split2(f.x, f.y, hi.x, lo.x);
-    split2(f.z, f.w, hi.y, lo.y);
-    *reinterpret_cast<uint2*>(sh + d * kTcVp + c) = hi;
-    *reinterpret_cast<uint2*>(sl + d * kTcVp + c) = lo;
-  }
-  __syncthreads();
-  if (warp * 16 >= tl.nb) return;  // no rows for this warp (no barrier follows)
-
   const uint32_t sqh = smem_u32(qh), sql = smem_u32(ql), skh = smem_u32(kh), skl = smem_u32(kl), svh = smem_u32(vh), svl = smem_u32(vl),
                  ssh = smem_u32(sh), ssl = smem_u32(sl);
   const int mi = lane >> 3, r8 = lane & 7, gq = lane >> 2, t4 = lane & 3;
   const int trow[2] = {warp * 16 + gq, warp * 16 + gq + 8};
-  const float* Cr = gated ? C + (warp * 16 - 1) * DP : nullptr;  // the reference row (before the warp's first; warp 0: zeros)
-
-  // does the block's own decay leave the range in which it can be multiplied in?
-  bool direct = false;
-  if constexpr (gated) {
-    float worst = 0.f;
-    for (int d = lane; d < D; d += 32) worst = fmaxf(worst, (warp > 0 ? Cr[d] : 0.f) - C[(warp * 16 + 15) * DP + d]);
-    direct = warp_max(worst) > kSafeLog2;
-  }
-
   float acc[8][4];   // S_in^T q, then everything
   float g[4][2][4];  // scores: key block j, key octet, fragment
 #pragma unroll
@@ -311,88 +330,147 @@ linattn_tc_out_kernel(const bf16* __restrict__ proj, const float* __restrict__ l
 #pragma unroll
     for (int n = 0; n < 2; ++n) g[j][n][0] = g[j][n][1] = g[j][n][2] = g[j][n][3] = 0.f;
 
-  for (int kk = 0; kk < D / 16; ++kk) {
-    uint32_t ah[4], al[4];     // the rows' operand of the state product
-    uint32_t gh[4], gl[4];     // ... and of the scores
-    float2 cr[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
-    const uint32_t aoff = ((warp * 16 + (mi & 1) * 8 + r8) * DP + kk * 16 + (mi >> 1) * 8) * 2;
-    ldmatrix_x4(ah, sqh + aoff);
+  const float* Sp = scr_u + (((size_t)blockIdx.x * a.H + h) * D) * a.V + v0;
+  const bool alq = raw_aligned(proj, a.ldp, a.q_off + h * D), alk = raw_aligned(proj, a.ldp, a.k_off + h * D);
+  for (int d0 = 0; d0 < D; d0 += kTcDc) {
+    const int nd = min(kTcDc, D - d0);
+    if (d0) __syncthreads();  // the previous pass's blocks have been used
     if constexpr (gated) {
-      // fragment x: row trow[x & 1], channels kk*16 + (x >> 1)*8 + 2 t4 and the next
-      if (warp > 0) {
-        cr[0] = *reinterpret_cast<const float2*>(Cr + kk * 16 + 2 * t4);
-        cr[1] = *reinterpret_cast<const float2*>(Cr + kk * 16 + 8 + 2 * t4);
-      }
-#pragma unroll
-      for (int x = 0; x < 4; ++x) {
-        const float2 c = *reinterpret_cast<const float2*>(C + trow[x & 1] * DP + kk * 16 + (x >> 1) * 8 + 2 * t4);
-        const float2 r = cr[x >> 1];
-        const float u = bf_lo(ah[x]), v = bf_hi(ah[x]);
-        split2(u * ex2_ftz(c.x - r.x), v * ex2_ftz(c.y - r.y), gh[x], gl[x]);
-        split2(u * ex2_ftz(c.x), v * ex2_ftz(c.y), ah[x], al[x]);
-      }
+      stage_raw(proj + tl.row0 * a.ldp + a.q_off + h * D + d0, a.ldp, tl, nd, alq, qh);
+      stage_raw(proj + tl.row0 * a.ldp + a.k_off + h * D + d0, a.ldp, tl, nd, alk, kh);
     } else {
-      ldmatrix_x4(al, sql + aoff);
-#pragma unroll
-      for (int x = 0; x < 4; ++x) { gh[x] = ah[x]; gl[x] = al[x]; }
+      const size_t at = tl.row0 * C + h * D + d0;
+      stage_raw(hi + at, C, tl, nd, true, qh);
+      stage_raw(lo + at, C, tl, nd, true, ql);
+      stage_raw(hi + at + a.H * D, C, tl, nd, true, kh);
+      stage_raw(lo + at + a.H * D, C, tl, nd, true, kl);
     }
+    cp_async_commit();
+    if constexpr (gated) {
+      // two threads per channel: rows 0..31, and rows 32..63 after the first half's total
+      const int d = tid & 63, part = tid >> 6;
+      const bool ok = d < nd;
+      const float* lp = lg + tl.row0 * ((size_t)a.H * D) + h * D + d0 + d;
+      float c = 0.f;
+      if (part == 1 && ok)
+        for (int t = 0; t < min(32, tl.nb); ++t) c += lp[(size_t)t * a.H * D] * kLog2e;
+      for (int t0 = part * 32; t0 < part * 32 + 32; t0 += 8) {
+        float l8[8];
 #pragma unroll
-    for (int jp = 0; jp < 4; ++jp) {
-      uint32_t bh[4], bl[4];
-      const uint32_t soff = ((kk * 16 + (mi & 1) * 8 + r8) * kTcVp + jp * 16 + (mi >> 1) * 8) * 2;
-      ldmatrix_x4_trans(bh, ssh + soff);
-      ldmatrix_x4_trans(bl, ssl + soff);
-      mma_16816(acc[2 * jp], ah, bh[0], bh[1]);
-      mma_16816(acc[2 * jp + 1], ah, bh[2], bh[3]);
-      mma_16816(acc[2 * jp], ah, bl[0], bl[1]);
-      mma_16816(acc[2 * jp + 1], ah, bl[2], bl[3]);
-      mma_16816(acc[2 * jp], al, bh[0], bh[1]);
-      mma_16816(acc[2 * jp + 1], al, bh[2], bh[3]);
+        for (int u = 0; u < 8; ++u) l8[u] = ok && t0 + u < tl.nb ? lp[(size_t)(t0 + u) * a.H * D] * kLog2e : 0.f;
+#pragma unroll
+        for (int u = 0; u < 8; ++u) { c += l8[u]; Cs[(t0 + u) * kTcDp + d] = c; }
+      }
     }
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      if (j > warp || (j == warp && direct)) continue;
-      uint32_t bh[4], bl[4];
-      const uint32_t koff = ((j * 16 + (mi >> 1) * 8 + r8) * DP + kk * 16 + (mi & 1) * 8) * 2;
-      ldmatrix_x4(bh, skh + koff);
+    for (int i = tid; i < kTcDc * (kTcVc / 4); i += kTcThreads) {
+      const int d = i / (kTcVc / 4), c = 4 * (i % (kTcVc / 4));
+      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < nv && d < nd) f = *reinterpret_cast<const float4*>(Sp + (size_t)(d0 + d) * a.V + c);
+      uint2 fh, fl;
+      split2(f.x, f.y, fh.x, fl.x);
+      split2(f.z, f.w, fh.y, fl.y);
+      *reinterpret_cast<uint2*>(sh + d * kTcVp + c) = fh;
+      *reinterpret_cast<uint2*>(sl + d * kTcVp + c) = fl;
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    if (warp * 16 >= tl.nb) continue;  // no rows for this warp
+    // gated: the reference row of the warp's scores (the one before its first; warp 0: zeros), and whether its own block's
+    // decay in this pass's channels leaves the range in which it can be multiplied in
+    const float* Cr = Cs + (warp > 0 ? warp * 16 - 1 : 0) * kTcDp;
+    bool direct = false;
+    if constexpr (gated) {
+      float worst = 0.f;
+      for (int d = lane; d < nd; d += 32) worst = fmaxf(worst, (warp > 0 ? Cr[d] : 0.f) - Cs[(warp * 16 + 15) * kTcDp + d]);
+      direct = warp_max(worst) > kSafeLog2;
+    }
+    for (int kk = 0; kk < nd / 16; ++kk) {
+      uint32_t ah[4], al[4];     // the rows' operand of the state product
+      uint32_t gh[4], gl[4];     // ... and of the scores
+      float2 cr[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
+      const uint32_t aoff = ((warp * 16 + (mi & 1) * 8 + r8) * kTcDp + kk * 16 + (mi >> 1) * 8) * 2;
+      ldmatrix_x4(ah, sqh + aoff);
       if constexpr (gated) {
-        // fragment x: key row j*16 + (x >> 1)*8 + gq, channels kk*16 + (x & 1)*8 + 2 t4 and the next
+        // fragment x: row trow[x & 1], channels kk*16 + (x >> 1)*8 + 2 t4 and the next
+        if (warp > 0) {
+          cr[0] = *reinterpret_cast<const float2*>(Cr + kk * 16 + 2 * t4);
+          cr[1] = *reinterpret_cast<const float2*>(Cr + kk * 16 + 8 + 2 * t4);
+        }
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
-          const float2 c = *reinterpret_cast<const float2*>(C + (j * 16 + (x >> 1) * 8 + gq) * DP + kk * 16 + (x & 1) * 8 + 2 * t4);
-          const float2 r = cr[x & 1];
-          split2(bf_lo(bh[x]) * ex2_ftz(r.x - c.x), bf_hi(bh[x]) * ex2_ftz(r.y - c.y), bh[x], bl[x]);
+          const float2 c = *reinterpret_cast<const float2*>(Cs + trow[x & 1] * kTcDp + kk * 16 + (x >> 1) * 8 + 2 * t4);
+          const float2 r = cr[x >> 1];
+          const float u = bf_lo(ah[x]), v = bf_hi(ah[x]);
+          split2(u * ex2_ftz(c.x - r.x), v * ex2_ftz(c.y - r.y), gh[x], gl[x]);
+          split2(u * ex2_ftz(c.x), v * ex2_ftz(c.y), ah[x], al[x]);
         }
       } else {
-        ldmatrix_x4(bl, skl + koff);
+        ldmatrix_x4(al, sql + aoff);
+#pragma unroll
+        for (int x = 0; x < 4; ++x) { gh[x] = ah[x]; gl[x] = al[x]; }
       }
-      mma_16816(g[j][0], gh, bh[0], bh[1]);
-      mma_16816(g[j][1], gh, bh[2], bh[3]);
-      mma_16816(g[j][0], gh, bl[0], bl[1]);
-      mma_16816(g[j][1], gh, bl[2], bl[3]);
-      mma_16816(g[j][0], gl, bh[0], bh[1]);
-      mma_16816(g[j][1], gl, bh[2], bh[3]);
-    }
-  }
-  const float l2 = gated ? 0.f : a.log_decay[h] * kLog2e;
-  if constexpr (gated) {
-    if (direct) {
+#pragma unroll
+      for (int jp = 0; jp < 4; ++jp) {
+        uint32_t bh[4], bl[4];
+        const uint32_t soff = ((kk * 16 + (mi & 1) * 8 + r8) * kTcVp + jp * 16 + (mi >> 1) * 8) * 2;
+        ldmatrix_x4_trans(bh, ssh + soff);
+        ldmatrix_x4_trans(bl, ssl + soff);
+        mma_16816(acc[2 * jp], ah, bh[0], bh[1]);
+        mma_16816(acc[2 * jp + 1], ah, bh[2], bh[3]);
+        mma_16816(acc[2 * jp], ah, bl[0], bl[1]);
+        mma_16816(acc[2 * jp + 1], ah, bl[2], bl[3]);
+        mma_16816(acc[2 * jp], al, bh[0], bh[1]);
+        mma_16816(acc[2 * jp + 1], al, bh[2], bh[3]);
+      }
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        if (j != warp) continue;
-#pragma unroll
-        for (int n = 0; n < 2; ++n)
+        if (j > warp || (j == warp && direct)) continue;
+        uint32_t bh[4], bl[4];
+        const uint32_t koff = ((j * 16 + (mi >> 1) * 8 + r8) * kTcDp + kk * 16 + (mi & 1) * 8) * 2;
+        ldmatrix_x4(bh, skh + koff);
+        if constexpr (gated) {
+          // fragment x: key row j*16 + (x >> 1)*8 + gq, channels kk*16 + (x & 1)*8 + 2 t4 and the next
 #pragma unroll
           for (int x = 0; x < 4; ++x) {
-            const int t = trow[x >> 1], s = j * 16 + n * 8 + 2 * t4 + (x & 1);
-            float u = 0.f;
-            if (s <= t)
-              for (int d = 0; d < D; ++d)
-                u = fmaf(__bfloat162float(qh[t * DP + d]) * __bfloat162float(kh[s * DP + d]), ex2_ftz(C[t * DP + d] - C[s * DP + d]), u);
-            g[j][n][x] = u;
+            const float2 c = *reinterpret_cast<const float2*>(Cs + (j * 16 + (x >> 1) * 8 + gq) * kTcDp + kk * 16 + (x & 1) * 8 + 2 * t4);
+            const float2 r = cr[x & 1];
+            split2(bf_lo(bh[x]) * ex2_ftz(r.x - c.x), bf_hi(bh[x]) * ex2_ftz(r.y - c.y), bh[x], bl[x]);
           }
+        } else {
+          ldmatrix_x4(bl, skl + koff);
+        }
+        mma_16816(g[j][0], gh, bh[0], bh[1]);
+        mma_16816(g[j][1], gh, bh[2], bh[3]);
+        mma_16816(g[j][0], gh, bl[0], bl[1]);
+        mma_16816(g[j][1], gh, bl[2], bl[3]);
+        mma_16816(g[j][0], gl, bh[0], bh[1]);
+        mma_16816(g[j][1], gl, bh[2], bh[3]);
       }
     }
+    if constexpr (gated) {
+      if (direct) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          if (j != warp) continue;
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+              const int t = trow[x >> 1], s = j * 16 + n * 8 + 2 * t4 + (x & 1);
+              float u = 0.f;
+              if (s <= t)
+                for (int d = 0; d < nd; ++d)
+                  u = fmaf(__bfloat162float(qh[t * kTcDp + d]) * __bfloat162float(kh[s * kTcDp + d]),
+                           ex2_ftz(Cs[t * kTcDp + d] - Cs[s * kTcDp + d]), u);
+              g[j][n][x] += u;
+            }
+        }
+      }
+    }
+  }  // passes over the key channels
+  if (warp * 16 >= tl.nb) return;
+  const float l2 = gated ? 0.f : a.log_decay[h] * kLog2e;
+  if constexpr (gated) {
 #pragma unroll
     for (int i = 0; i < 8; ++i)
 #pragma unroll
@@ -447,37 +525,52 @@ linattn_tc_out_kernel(const bf16* __restrict__ proj, const float* __restrict__ l
   }
 }
 
-template <bool gated>
-static int tc_local(const void* proj, const float* lg, const LinAttn& a, const int32_t* tiles, int n_tiles, float* scr_u, float* scr_w,
-                    cudaStream_t s) {
-  static PerDeviceOnce once;
-  DLI_ONCE_PER_DEVICE(once, dev, DLI_CUDA_CALL(cudaFuncSetAttribute(linattn_tc_local_kernel<gated>,
-                                                                     cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024)));
-  DLI_LAUNCH("linattn_tc_local", linattn_tc_local_kernel<gated>, dim3(n_tiles, a.H, (a.V + kTcVc - 1) / kTcVc), dim3(kTcThreads),
-             tc_local_smem(a.D, gated), s, (const bf16*)proj, lg, a, tiles, scr_u, scr_w);
+// fixed decay: the prepared rows in `prep` (hi rows, then lo rows; 2HD + HV floats' worth of bf16 pairs per row)
+static LinPrep prep_rows(float* prep, const LinAttn& a, int rows, const int32_t* tiles) {
+  bf16* hi = reinterpret_cast<bf16*>(prep);
+  return LinPrep{a.ent, tiles, hi, hi + (size_t)rows * a.H * (2 * a.D + a.V)};
+}
+
+static int tc_prep(const void* proj, const LinAttn& a, const LinPrep& p, int n_tiles, cudaStream_t s) {
+  const int half = a.rd / 2;
+  const bool wide = half % 8 == 0 && (a.D - a.rd) % 8 == 0 && a.D % 8 == 0 && a.V % 8 == 0 && a.ldp % 8 == 0 && a.q_off % 8 == 0 &&
+                    a.k_off % 8 == 0 && a.v_off % 8 == 0 && aligned16(proj) && aligned16(p.hi);
+  const dim3 grid(n_tiles, kLaTile / 8);
+  if (wide) DLI_LAUNCH("linattn_prep", linattn_prep_kernel<8>, grid, dim3(256), 0, s, (const bf16*)proj, a, p);
+  else DLI_LAUNCH("linattn_prep", linattn_prep_kernel<1>, grid, dim3(256), 0, s, (const bf16*)proj, a, p);
   return DLI_OK;
 }
 
-template <bool gated>
-static int tc_out(const void* proj, const float* lg, float* o, const LinAttn& a, const int32_t* tiles, int n_tiles, const float* scr_u,
-                  cudaStream_t s) {
-  static PerDeviceOnce once;
-  DLI_ONCE_PER_DEVICE(once, dev, DLI_CUDA_CALL(cudaFuncSetAttribute(linattn_tc_out_kernel<gated>,
-                                                                     cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024)));
-  DLI_LAUNCH("linattn_tc_out", linattn_tc_out_kernel<gated>, dim3(n_tiles, a.H, (a.V + kTcVc - 1) / kTcVc), dim3(kTcThreads),
-             tc_out_smem(a.D, gated), s, (const bf16*)proj, lg, o, a, tiles, scr_u);
-  return DLI_OK;
-}
+#define TC_LAUNCH(KERNEL, SMEM, ...)                                                                                      \
+  do {                                                                                                                    \
+    static PerDeviceOnce once;                                                                                            \
+    DLI_ONCE_PER_DEVICE(once, dev, DLI_CUDA_CALL(cudaFuncSetAttribute(KERNEL, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                                                       (int)(SMEM))));                                    \
+    DLI_LAUNCH(#KERNEL, KERNEL, dim3(n_tiles, a.H, (a.V + kTcVc - 1) / kTcVc), dim3(kTcThreads), SMEM, s, __VA_ARGS__);     \
+  } while (0)
 
-int linattn_tc_local(const void* proj, const float* lg, const LinAttn& a, const int32_t* tiles, int n_tiles, float* scr_u,
+int linattn_tc_local(const void* proj, float* row_scr, const LinAttn& a, int rows, const int32_t* tiles, int n_tiles, float* scr_u,
                      float* scr_w, cudaStream_t s) {
-  return a.log_decay ? tc_local<false>(proj, lg, a, tiles, n_tiles, scr_u, scr_w, s)
-                     : tc_local<true>(proj, lg, a, tiles, n_tiles, scr_u, scr_w, s);
+  if (a.log_decay) {
+    const LinPrep p = prep_rows(row_scr, a, rows, tiles);
+    const int rc = tc_prep(proj, a, p, n_tiles, s);
+    if (rc != DLI_OK) return rc;
+    TC_LAUNCH(linattn_tc_local_kernel<false>, tc_local_smem(false), (const bf16*)proj, p.hi, p.lo, nullptr, a, tiles, scr_u, scr_w);
+  } else {
+    TC_LAUNCH(linattn_tc_local_kernel<true>, tc_local_smem(true), (const bf16*)proj, nullptr, nullptr, row_scr, a, tiles, scr_u, scr_w);
+  }
+  return DLI_OK;
 }
 
-int linattn_tc_out(const void* proj, const float* lg, float* o, const LinAttn& a, const int32_t* tiles, int n_tiles,
+int linattn_tc_out(const void* proj, float* row_scr, float* o, const LinAttn& a, int rows, const int32_t* tiles, int n_tiles,
                    const float* scr_u, cudaStream_t s) {
-  return a.log_decay ? tc_out<false>(proj, lg, o, a, tiles, n_tiles, scr_u, s) : tc_out<true>(proj, lg, o, a, tiles, n_tiles, scr_u, s);
+  if (a.log_decay) {
+    const LinPrep p = prep_rows(row_scr, a, rows, tiles);
+    TC_LAUNCH(linattn_tc_out_kernel<false>, tc_out_smem(false), (const bf16*)proj, p.hi, p.lo, nullptr, o, a, tiles, scr_u);
+  } else {
+    TC_LAUNCH(linattn_tc_out_kernel<true>, tc_out_smem(true), (const bf16*)proj, nullptr, nullptr, row_scr, o, a, tiles, scr_u);
+  }
+  return DLI_OK;
 }
 
 }  // namespace dli

@@ -960,7 +960,7 @@ def linattn_ragged(proj, S, o, ent, H, D, V, q_off, k_off, v_off, silu=False, q_
     """Linear attention with a decaying matrix state over the rows of every entry; S float32 [slots, H, D, V] is advanced; o
     float32 [rows, H*V].  log_decay float32 [H]: fixed decay per head; else a decay per key channel from columns a_off.. of
     proj through a2 [H*D, rank], a2_b [H*D] (float32) and inv_tau.  blocked: small matrix products (steps with portions of
-    prompts; lg float32 scratch [rows, H*D] for a decay per channel), with tiles and scratch of linattn_scratch_floats(...)
+    prompts; lg float32 scratch, [rows, H*D] for a decay per channel, else [rows, 2*H*D + H*V] for the tensor cores), with tiles and scratch of linattn_scratch_floats(...)
     floats all 64-row tiles in parallel (on the tensor cores where linattn_tc_supported)."""
     _req(proj, proj.dtype), _f32(S, o, cos_t, sin_t, log_decay, a2, a2_b, lg, scratch), _i32(ent, tiles)
     rows, n_ent = proj.shape[0], ent.numel() // 4
@@ -969,9 +969,11 @@ def linattn_ragged(proj, S, o, ent, H, D, V, q_off, k_off, v_off, silu=False, q_
     par = bool(blocked) and scratch is not None and n_tiles > 0
     if par and scratch.numel() < linattn_scratch_floats(n_tiles, H, D, V):
         raise ValueError("linattn_ragged: scratch too small")
-    if o.numel() < rows * H * V or (gated and blocked and lg.numel() < rows * H * D):
+    if o.numel() < rows * H * V or (blocked and gated and lg.numel() < rows * H * D) or \
+            (blocked and not gated and lg is not None and lg.numel() < rows * H * (2 * D + V)):
         raise ValueError("linattn_ragged: output or log-decay scratch too small")
-    _call("dli_linattn_ragged", (3 if par else 1) + int(gated and bool(blocked)), _p(proj), _p(S), _p(o), _p(ent), n_ent, rows, H, D,
+    tc = par and lg is not None and linattn_tc_supported(D, V, gated, silu, rd, proj.dtype)
+    _call("dli_linattn_ragged", (3 if par else 1) + int(bool(blocked) and (gated or tc)), _p(proj), _p(S), _p(o), _p(ent), n_ent, rows, H, D,
           V, proj.shape[1], int(q_off), int(k_off), int(v_off), int(bool(silu)), float(q_scale), float(k_scale), _p(cos_t),
           _p(sin_t), int(rd), _p(log_decay), int(a_off), a2.shape[1] if a2 is not None else 0, _p(a2), _p(a2_b), float(inv_tau),
           int(bool(blocked)), _p(lg), _p(tiles) if par else None, n_tiles if par else 0, _p(scratch) if par else None, _dt(proj),

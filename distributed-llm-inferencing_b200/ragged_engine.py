@@ -594,9 +594,10 @@ class RaggedEngine:
         if sides:
             self._sg = torch.empty(rows * max(sides), dtype=E, device=dev)
             self._sa = torch.empty(rows * max(sides), dtype=E, device=dev)
-        gated = [m.heads * m.dim for m in mx if m.kind == "linear_attention" and m.tau]
-        if gated:
-            self._lg = torch.empty(rows * max(gated), dtype=f32, device=dev)  # log decays per row and key channel
+        lin = [m.heads * m.dim if m.tau else m.heads * (2 * m.dim + m.vdim) for m in mx if m.kind == "linear_attention"]
+        if lin:
+            # per row: log decays of every key channel, or the prepared q | k | v
+            self._lg = torch.empty(rows * max(lin), dtype=f32, device=dev)
         if s.streams:
             self._xst = torch.empty(s.streams, rows, s.width, dtype=f32, device=dev)
         if any(L.parallel or L.pre_norm for L in s.layers):
@@ -1142,7 +1143,7 @@ class RaggedEngine:
                            q_scale=m.q_scale, k_scale=m.k_scale, cos_t=cos_t, sin_t=sin_t, rd=m.rot_dims,
                            log_decay=P["log_decay"], a_off=off["a"], a2=P["a2"], a2_b=P["a2_b"],
                            inv_tau=1.0 / m.tau if m.tau else 1.0, blocked=long_step,
-                           lg=self._lg[:rows * H * D] if m.tau else None, tiles=d_tiles if scr is not None else None, scratch=scr)
+                           lg=self._lg[:rows * (H * D if m.tau else H * (2 * D + V))], tiles=d_tiles if scr is not None else None, scratch=scr)
         n_h, n_v = (1, H * V) if m.norm_heads_together else (H, V)
         ops.head_rmsnorm_gate(o, proj, P["out_norm"], mix, n_h, n_v, self.spec.eps, gate=1 if m.gate_fn == "silu" else 2,
                               g_off=off["g"])

@@ -660,7 +660,8 @@ int dli_streams_close(const void* y, float* x, size_t xs_stride, int n_streams, 
  * rotated in pairs (i, i + rd/2) (cos_t / sin_t [positions, rd/2]); q_scale / k_scale: factors.  The decay is
  * exp(log_decay[h]), or, with log_decay NULL, per key channel sigmoid(a2 . proj[row, a_off : +rank] + a2_b)^inv_tau
  * (a2 [H*D, rank], a2_b [H*D] fp32).  blocked != 0 (steps with portions of prompts): 16 rows at a time as small matrix
- * products, else row by row; lg: scratch [rows, H*D] for the blocked form with a decay per channel; with tiles (as for
+ * products, else row by row; lg: scratch of the blocked form, [rows, H*D] with a decay per
+ * channel, else [rows, 2*H*D + H*V] for the tensor-core form (NULL: not used); with tiles (as for
  * dli_attn_ragged_tc) and scratch of dli_linattn_scratch_floats floats the 64-row tiles of all entries run in parallel, on
  * the tensor cores where dli_linattn_tc_supported (bf16 rows; operands that are not exact in bf16 as the sum of two). */
 int dli_linattn_tc_supported(int D, int V, int gated, int silu, int rd, int dt);
