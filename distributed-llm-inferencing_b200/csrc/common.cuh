@@ -188,16 +188,40 @@ __device__ __forceinline__ float gelu_new_f(float x) {
   const float k = 0.7978845608028654f;  // sqrt(2/pi)
   return 0.5f * x * (1.0f + tanhf(k * (x + 0.044715f * x * x * x)));
 }
+// The tanh form of gelu at silu's cost: 0.5 (1 + tanh z) = 1 / (1 + e^(-2z)).
+__device__ __forceinline__ float gelu_gate(float x) {
+  return x / (1.0f + expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
+}
 // Epilogue of a gated projection pair.  act == NULL: silu(gate) * up with the rounding points of a bf16 framework.
 // act = {limit, alpha} (two floats on the device): the clamped form g * sigmoid(alpha g) * (u + 1) with
 // g = min(gate, limit), u = clamp(up, -limit, limit); limit <= 0: gelu (tanh form) of the gate, times up.
 __device__ __forceinline__ float gated_combine(float gte, float up, const float* __restrict__ act) {
   if (act == nullptr) return round_bf16(silu_f(gte)) * up;
   const float lim = act[0], alpha = act[1];
-  // 0.5 (1 + tanh z) = 1 / (1 + e^(-2z)): the tanh form of gelu at silu's cost
-  if (lim <= 0.f) return gte / (1.0f + expf(-1.5957691216057308f * (gte + 0.044715f * gte * gte * gte))) * up;
+  if (lim <= 0.f) return gelu_gate(gte) * up;
   const float g = fminf(gte, lim), u = fminf(fmaxf(up, -lim), lim);
   return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+}
+
+// The same on N gates (in place) and N ups: one test of the form for all of them.
+template <int N>
+__device__ __forceinline__ void gated_combine_n(float (&g)[N], const float (&u)[N], const float* __restrict__ act) {
+  if (act == nullptr) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) g[j] = gated_combine(g[j], u[j], nullptr);
+    return;
+  }
+  const float lim = act[0], alpha = act[1];
+  if (lim <= 0.f) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) g[j] = gelu_gate(g[j]) * u[j];
+  } else {
+#pragma unroll
+    for (int j = 0; j < N; ++j) {
+      const float c = fminf(g[j], lim), v = fminf(fmaxf(u[j], -lim), lim);
+      g[j] = c / (1.0f + expf(-alpha * c)) * (v + 1.0f);
+    }
+  }
 }
 
 }  // namespace dli

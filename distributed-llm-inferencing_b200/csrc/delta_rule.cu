@@ -470,14 +470,51 @@ head_rmsnorm_gate_kernel(const float* __restrict__ o, const E* __restrict__ proj
   const size_t row = item / a.H;
   const int h = (int)(item - row * a.H);
   const float* src = o + item * a.V;
-  float ss = 0.f;
-  for (int v = me * VEC; v < a.V; v += group * VEC) {
+  const E* gp = a.gate ? proj + row * a.ldp + a.g_off + h * a.V : nullptr;
+  const float* wp = w ? w + (a.w_heads ? h * a.V : 0) : nullptr;
+  E* dst = out + row * a.ldo + h * a.V;
+  auto ld_o = [&](int v, float (&f)[VEC]) {
     if constexpr (VEC == 4) {
-      const float4 f = *reinterpret_cast<const float4*>(src + v);
-      ss = fmaf(f.x, f.x, ss); ss = fmaf(f.y, f.y, ss); ss = fmaf(f.z, f.z, ss); ss = fmaf(f.w, f.w, ss);
+      const float4 u = *reinterpret_cast<const float4*>(src + v);
+      f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w;
     } else {
-      ss = fmaf(src[v], src[v], ss);
+      f[0] = src[v];
     }
+  };
+  auto ld_g = [&](int v, float (&z)[VEC]) {
+    if constexpr (VEC == 4 && sizeof(E) == 2) {
+      const uint2 u = *reinterpret_cast<const uint2*>(gp + v);
+      z[0] = bf_lo(u.x); z[1] = bf_hi(u.x); z[2] = bf_lo(u.y); z[3] = bf_hi(u.y);
+    } else if constexpr (VEC == 4) {
+      const float4 u = *reinterpret_cast<const float4*>(gp + v);
+      z[0] = u.x; z[1] = u.y; z[2] = u.z; z[3] = u.w;
+    } else {
+      z[0] = d_to_f(gp[v]);
+    }
+  };
+  // the first kKeep pieces of a thread stay in registers, and their loads are all in flight before the reduction
+  constexpr int kKeep = 4;
+  float f[kKeep][VEC], z[kKeep][VEC];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int v = (me + i * group) * VEC;
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) f[i][k] = z[i][k] = 0.f;
+    if (v < a.V) {
+      ld_o(v, f[i]);
+      if (a.gate) ld_g(v, z[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i)
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) ss = fmaf(f[i][k], f[i][k], ss);
+  for (int v = (me + kKeep * group) * VEC; v < a.V; v += group * VEC) {
+    float t[VEC];
+    ld_o(v, t);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) ss = fmaf(t[k], t[k], ss);
   }
   ss = warp_sum(ss);
   if (kWide) {
@@ -487,40 +524,40 @@ head_rmsnorm_gate_kernel(const float* __restrict__ o, const E* __restrict__ proj
     for (int i = 0; i < (int)(blockDim.x >> 5); ++i) ss += red[i];
   }
   const float r = 1.f / sqrtf(ss / a.V + a.eps);
-  const E* gp = a.gate ? proj + row * a.ldp + a.g_off + h * a.V : nullptr;
-  const float* wp = w ? w + (a.w_heads ? h * a.V : 0) : nullptr;
-  E* dst = out + row * a.ldo + h * a.V;
-  auto gated = [&](float y, float z) {
-    return a.gate == 1 ? y * (z / (1.f + expf(-z))) : y / (1.f + expf(-z));
-  };
-  for (int v = me * VEC; v < a.V; v += group * VEC) {
-    if constexpr (VEC == 4) {
-      const float4 f = *reinterpret_cast<const float4*>(src + v);
-      float y[4] = {f.x * r, f.y * r, f.z * r, f.w * r};
-      if (wp) {
-        const float4 w4 = *reinterpret_cast<const float4*>(wp + v);
-        y[0] *= w4.x; y[1] *= w4.y; y[2] *= w4.z; y[3] *= w4.w;
-      }
-      if (a.gate) {
-        float z[4];
-        if constexpr (sizeof(E) == 2) {
-          const uint2 u = *reinterpret_cast<const uint2*>(gp + v);
-          z[0] = bf_lo(u.x); z[1] = bf_hi(u.x); z[2] = bf_lo(u.y); z[3] = bf_hi(u.y);
-        } else {
-          const float4 z4 = *reinterpret_cast<const float4*>(gp + v);
-          z[0] = z4.x; z[1] = z4.y; z[2] = z4.z; z[3] = z4.w;
-        }
+  auto finish = [&](int v, float (&y)[VEC], const float (&zz)[VEC]) {
+    float wv[VEC];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) y[i] = gated(y[i], z[i]);
+    for (int k = 0; k < VEC; ++k) wv[k] = 1.f;
+    if (wp) {
+      if constexpr (VEC == 4) {
+        const float4 w4 = *reinterpret_cast<const float4*>(wp + v);
+        wv[0] = w4.x; wv[1] = w4.y; wv[2] = w4.z; wv[3] = w4.w;
+      } else {
+        wv[0] = wp[v];
       }
-      if constexpr (sizeof(E) == 2) *reinterpret_cast<uint2*>(dst + v) = make_uint2(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]));
-      else *reinterpret_cast<float4*>(dst + v) = make_float4(y[0], y[1], y[2], y[3]);
-    } else {
-      float y = src[v] * r;
-      if (wp) y *= wp[v];
-      if (a.gate) y = gated(y, d_to_f(gp[v]));
-      dst[v] = d_from_f<E>(y);
     }
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) {
+      y[k] = y[k] * r * wv[k];
+      if (a.gate == 1) y[k] *= zz[k] / (1.f + expf(-zz[k]));
+      else if (a.gate == 2) y[k] /= 1.f + expf(-zz[k]);
+    }
+    if constexpr (VEC == 4 && sizeof(E) == 2) *reinterpret_cast<uint2*>(dst + v) = make_uint2(pack_bf16(y[0], y[1]), pack_bf16(y[2], y[3]));
+    else if constexpr (VEC == 4) *reinterpret_cast<float4*>(dst + v) = make_float4(y[0], y[1], y[2], y[3]);
+    else dst[v] = d_from_f<E>(y[0]);
+  };
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) {
+    const int v = (me + i * group) * VEC;
+    if (v < a.V) finish(v, f[i], z[i]);
+  }
+  for (int v = (me + kKeep * group) * VEC; v < a.V; v += group * VEC) {
+    float t[VEC], zz[VEC];
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) zz[k] = 0.f;
+    ld_o(v, t);
+    if (a.gate) ld_g(v, zz);
+    finish(v, t, zz);
   }
 }
 

@@ -180,11 +180,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]);
           if (kGated) {
+            float up[16];
 #pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              const float gte = round_bf16(v[j]), up = round_bf16(__uint_as_float(r2[j]));
-              v[j] = gated_combine(gte, up, kGated ? reinterpret_cast<const float*>(bias) : nullptr);
-            }
+            for (int j = 0; j < 16; ++j) { v[j] = round_bf16(v[j]); up[j] = round_bf16(__uint_as_float(r2[j])); }
+            gated_combine_n(v, up, reinterpret_cast<const float*>(bias));
           } else {
             if (epilogue & DLI_EPI_BIAS) {
 #pragma unroll
@@ -664,11 +663,10 @@ gemm_prefill_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
 #pragma unroll
           for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]);
           if (kGated) {
+            float up[16];
 #pragma unroll
-            for (int j = 0; j < 16; ++j) {
-              const float gte = round_bf16(v[j]), up = round_bf16(__uint_as_float(r2[j]));
-              v[j] = gated_combine(gte, up, kGated ? reinterpret_cast<const float*>(bias) : nullptr);
-            }
+            for (int j = 0; j < 16; ++j) { v[j] = round_bf16(v[j]); up[j] = round_bf16(__uint_as_float(r2[j])); }
+            gated_combine_n(v, up, reinterpret_cast<const float*>(bias));
           } else {
             if (epilogue & DLI_EPI_BIAS) {
 #pragma unroll

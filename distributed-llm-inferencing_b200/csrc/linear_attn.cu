@@ -249,13 +249,19 @@ linattn_blocks_kernel(const E* __restrict__ proj, const float* __restrict__ lg, 
     int n_own = 0;
     for (int d = tid; d < D; d += 256, ++n_own) {
       if (gated) {
+        // c_L - c_t as the sum of the later rows' logarithms: a difference of running sums would lose the small ones
+        // behind a fast decay
+        float r = 0.f;
+        for (int t = kLaL - 1; t >= 0; --t) {
+          kT[d * kLaP + t] = ks[t * DP + d] * expf(r);
+          r += cs[t * DP + d];
+        }
+        if (mode == 1 && n_own < 4) total[n_own] += r;
         float c = 0.f;
-        for (int t = 0; t < kLaL; ++t) { c += cs[t * DP + d]; cs[t * DP + d] = c; }
-        if (mode == 1 && n_own < 4) total[n_own] += c;
         for (int t = 0; t < kLaL; ++t) {
-          const float ct = cs[t * DP + d];
-          if (mode != 1) qT[d * kLaP + t] = qs[t * DP + d] * expf(ct);
-          kT[d * kLaP + t] = ks[t * DP + d] * expf(c - ct);
+          c += cs[t * DP + d];
+          cs[t * DP + d] = c;
+          if (mode != 1) qT[d * kLaP + t] = qs[t * DP + d] * expf(c);
         }
       } else {
         for (int t = 0; t < kLaL; ++t) {

@@ -47,7 +47,7 @@ __global__ void __launch_bounds__(1024)
 embedding_f32_kernel(const int32_t* __restrict__ ids, const E* __restrict__ table, float* __restrict__ x,
                      float* __restrict__ x2, E* __restrict__ xe, int d, int vocab, float scale,
                      const int32_t* __restrict__ row_ent, const int32_t* __restrict__ ent,
-                     const float* __restrict__ inv_freq, BigramTab bg, int x_copies, size_t x_stride) {
+                     const float* __restrict__ inv_freq, BigramTab bg, int x_copies, size_t x_stride, int vec) {
   pdl_wait();
   pdl_trigger();
   const size_t row = blockIdx.x;
@@ -75,6 +75,33 @@ embedding_f32_kernel(const int32_t* __restrict__ ids, const E* __restrict__ tabl
       if (threadIdx.x == 0) bg.last[e.x] = ids[e.y + e.z - 1];
     }
     brow = reinterpret_cast<const E*>(bg.table) + (size_t)b * d;
+  }
+  if (!inv_freq && vec) {  // four channels per thread and access
+    for (int c = threadIdx.x * 4; c < d; c += blockDim.x * 4) {
+      float v[4], b[4] = {0.f, 0.f, 0.f, 0.f};
+      auto ld = [&](const E* p, float (&f)[4]) {
+        if constexpr (sizeof(E) == 2) {
+          const uint2 u = *reinterpret_cast<const uint2*>(p);
+          f[0] = bf_lo(u.x); f[1] = bf_hi(u.x); f[2] = bf_lo(u.y); f[3] = bf_hi(u.y);
+        } else {
+          const float4 u = *reinterpret_cast<const float4*>(p);
+          f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w;
+        }
+      };
+      ld(table + (size_t)id * d + c, v);
+      if (brow) ld(brow + c, b);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) v[k] = v[k] * scale + b[k];
+      const float4 o = make_float4(v[0], v[1], v[2], v[3]);
+      *reinterpret_cast<float4*>(x + row * d + c) = o;
+      for (int k = 1; k < x_copies; ++k) *reinterpret_cast<float4*>(x + k * x_stride + row * d + c) = o;
+      if (x2) *reinterpret_cast<float4*>(x2 + row * d + c) = o;
+      if (xe) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) xe[row * d + c + k] = from_f<E>(v[k]);
+      }
+    }
+    return;
   }
   for (int c = threadIdx.x; c < d; c += blockDim.x) {
     float v = to_f(table[(size_t)id * d + c]) * scale;
@@ -611,11 +638,14 @@ int dli_embedding_f32(const int32_t* ids, const void* table, float* x, float* x2
                 "dli_embedding_f32: a pair table needs its row count, the slots' last tokens, row_ent and a 16-byte aligned ent");
   DLI_CHECK_ARG(x_copies <= 1 || x_stride >= (size_t)rows * d, "dli_embedding_f32: copies of x overlap");
   const BigramTab bg{bigram, buckets, mul_prev, mul_cur, last};
+  const uintptr_t ea = (dt == 0 ? 8 : 16) - 1;
+  const int vec = d % 4 == 0 && ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(bigram)) & ea) == 0 && aligned16(x) &&
+                  aligned16(x2) && x_stride % 4 == 0;
   DT_CHECK(dt);
   if (rows <= 0) return DLI_OK;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (dt == 0) DLI_LAUNCH("embedding_f32", embedding_f32_kernel<bf16>, dim3(rows), dim3(row_threads(rows, d)), 0, s, ids, (const bf16*)table, x, x2, (bf16*)xe, d, vocab, scale, row_ent, ent, inv_freq, bg, x_copies, x_stride);
-  else DLI_LAUNCH("embedding_f32", embedding_f32_kernel<float>, dim3(rows), dim3(row_threads(rows, d)), 0, s, ids, (const float*)table, x, x2, (float*)xe, d, vocab, scale, row_ent, ent, inv_freq, bg, x_copies, x_stride);
+  if (dt == 0) DLI_LAUNCH("embedding_f32", embedding_f32_kernel<bf16>, dim3(rows), dim3(row_threads(rows, d)), 0, s, ids, (const bf16*)table, x, x2, (bf16*)xe, d, vocab, scale, row_ent, ent, inv_freq, bg, x_copies, x_stride, vec);
+  else DLI_LAUNCH("embedding_f32", embedding_f32_kernel<float>, dim3(rows), dim3(row_threads(rows, d)), 0, s, ids, (const float*)table, x, x2, (float*)xe, d, vocab, scale, row_ent, ent, inv_freq, bg, x_copies, x_stride, vec);
   return DLI_OK;
 }
 
