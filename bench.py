@@ -1197,16 +1197,21 @@ def salizen_kernel_times(eng, spec, T, peaks):
             H, D, V = m.heads, m.dim, m.vdim
             proj = (0.5 * torch.randn(rows, eng.layers[li]["w_proj"].shape[0], device=dev)).to(E)
             mix = torch.empty(rows, H * V, dtype=E, device=dev)
-            ms = timeit(lambda: eng._linear_attention(li, m, PP, proj, mix, rows, views, rows > 1), n=3, reps=5)
             o = torch.randn(rows, H * V, device=dev)
             nh, nv = (1, H * V) if m.norm_heads_together else (H, V)
             ms_n = timeit(lambda: ops.head_rmsnorm_gate(o, proj, PP["out_norm"], mix, nh, nv, 1e-6, gate=1, g_off=PP["off"]["g"]))
             put(f"{tag}_{name}_norm_gate", ms_n, byt=rows * H * V * (4 + 2 * eb))
             if rows > 1:
+                ms = timeit(lambda: eng._linear_attention(li, m, PP, proj, mix, rows, views, True), n=3, reps=5)
                 put(f"{tag}_{name}_recurrence", ms - ms_n, cuda_core=4 * rows * H * D * V)   # update and read-out of the state
                 res[f"{tag}_{name}_recurrence"]["of_hbm"] = round(rows * H * (2 * D * eb + V * (eb + 4)) / ((ms - ms_n) / 1e3) / hbm, 3)
             else:
-                put(f"{tag}_{name}_recurrence", ms - ms_n, byt=2 * H * D * V * 4)
+                of, rot = PP["off"], eng._table(m.rot_base, m.rot_dims, m.rot_scaling) if m.rot_dims else (None, None)
+                ms = timeit(lambda: ops.linattn_ragged(proj, eng.slots[("S", li)], o, ent, H, D, V, of["q"], of["k"], of["v"], silu=m.qkv_silu,
+                                                       q_scale=m.q_scale, k_scale=m.k_scale, cos_t=rot[0], sin_t=rot[1], rd=m.rot_dims,
+                                                       log_decay=PP["log_decay"], a_off=of["a"], a2=PP["a2"], a2_b=PP["a2_b"],
+                                                       inv_tau=1.0 / m.tau if m.tau else 1.0))
+                put(f"{tag}_{name}_recurrence", ms, byt=2 * H * D * V * 4)
         # windowed attention with soft cap, sink and a gate per channel; without the cap
         li = next(i for i, L in enumerate(spec.layers) if L.mixer.kind == "side_by_side")
         m, PP = spec.layers[li].mixer.parts[0], eng.layers[li]["parts"][0]
