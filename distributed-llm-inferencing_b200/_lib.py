@@ -79,17 +79,17 @@ SIGNATURES = {
     "dli_latent_prep": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _f, _vp, _vp,
                              _i, _i, _i, _vp]),
     "dli_latent_q_absorb": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp]),
-    "dli_latent_v_up": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp]),
+    "dli_latent_v_up": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp]),
     "dli_latent_expand": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp]),
     "dli_sigmoid_gate": (_i, [_vp, _vp, _i, _i, _i, _i, _i, _vp]),
     "dli_conv1d_act_ragged": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp]),
     "dli_ssm_scan_ragged": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _vp, _i, _vp]),
     "dli_ssm_parallel_scratch_floats": (_sz, [_i, _i, _i, _i]),
     "dli_gated_group_rmsnorm": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _i, _vp]),
-    "dli_moe_route": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp]),
+    "dli_moe_route": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _i, _vp, _vp, _vp]),
     "dli_moe_sel_supported": (_i, [_i, _i, _i, _i]),
-    "dli_moe_sel_bf16": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _f, _f, _i, _vp]),
-    "dli_moe_act": (_i, [_vp, _vp, _vp, _i, _i, _i, _f, _i, _f, _f, _i, _i, _i, _vp]),
+    "dli_moe_sel_bf16": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _f, _f, _i, _i, _vp, _vp]),
+    "dli_moe_act": (_i, [_vp, _vp, _vp, _i, _i, _i, _f, _i, _f, _f, _i, _i, _i, _i, _vp, _vp]),
     "dli_scalar_rmsnorm_f32": (_i, [_vp, _vp, _i, _i, _f, _f, _vp]),
     "dli_postnorm_add_norm": (_i, [_vp, _vp, _vp, _i, _i, _f, _f, _f, _i, _vp]),
     "dli_causal_conv_ragged": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp]),
@@ -98,7 +98,7 @@ SIGNATURES = {
     "dli_linear_any": (_i, [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp]),
     "dli_silu_mul": (_i, [_vp, _vp, _i, _i, _i, _i, _vp, _i, _vp]),
     "dli_attn_prep_append": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i,
-                                  _vp, _vp, _f, _vp, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _vp]),
+                                  _vp, _vp, _f, _vp, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _i, _vp]),
     "dli_attn_ragged": (_i, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _vp, _i,
                              _i, _vp, _vp, _i, _i, _vp, _i, _vp, _vp, _f, _i, _f, _i, _vp]),
     "dli_attn_ragged_tc_supported": (_i, [_i, _i, _i]),
@@ -115,6 +115,8 @@ SIGNATURES = {
     "dli_head_rmsnorm_gate": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _i, _i, _i, _i, _i, _vp]),
     "dli_streams_close": (_i, [_vp, _vp, _sz, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp, _vp, _vp, _vp, _vp, _vp,
                                _vp, _i, _i, _i, _i, _i, _f, _i, _vp]),
+    "dli_dyn_tanh_close": (_i, [_vp, _vp, _vp, _f, _f, _vp, _vp, _vp, _vp, _f, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp,
+                                _vp, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp, _vp]),
     "dli_linattn_tc_supported": (_i, [_i, _i, _i, _i, _i, _i]),
     "dli_linattn_scratch_floats": (_sz, [_i, _i, _i, _i]),
     "dli_linattn_ragged": (_i, [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _vp, _i, _vp, _i, _i,

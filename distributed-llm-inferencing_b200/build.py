@@ -38,6 +38,7 @@ SOURCES = [
     "delta_rule.cu",
     "prenorm_rows.cu",
     "stream_rows.cu",
+    "dyn_tanh_rows.cu",
     "linear_attn.cu",
     "linear_attn_tc.cu",
 ]

@@ -1,6 +1,7 @@
 // Attention over a paged cache for a RAGGED step (rows of several sequences, a prompt's portion beside single
 // decoded tokens), with the options a layer can switch on independently:
-//   - per-head RMS norm of queries and keys (one weight vector of the head size, shared by the heads),
+//   - per-head RMS norm of queries and keys (one weight vector of the head size, shared by the heads), or one norm over
+//     the whole query / key projection (a weight per row of it),
 //   - rotary positions on the first `rd` dimensions, INTERLEAVED pairs (2i, 2i+1), angles from a host-made fp32
 //     cos/sin table [positions, rd/2] (so any frequency scaling is the table's business),
 //   - rotated values: the value of position j is turned by j over all its pairs before it is cached, and a
@@ -51,7 +52,31 @@ struct AttnPrep {
   const float* bias;        // [>= the projection's q / k / v columns] fp32 or NULL: added to the projection's columns
   int q_only;               // 1: only the queries are made; keys and values are another layer's
   int halves;               // rotation pairs: 0: (2i, 2i+1), 1: (i, i + rd/2)
+  int whole;                // 1: the norms run over all heads at once, qn [H*D] and kn [G*D]
 };
+
+// this thread's part of the sum of squares of n consecutive columns (+ bias): 16-byte loads where their start allows
+template <typename E>
+__device__ __forceinline__ float prep_sum_squares(const E* src, const float* bs, int n) {
+  constexpr int V = 16 / (int)sizeof(E);
+  float ss = 0.f;
+  int c0 = 0;
+  if (!bs && (reinterpret_cast<uintptr_t>(src) & 15u) == 0) {
+    c0 = n / V * V;
+    for (int c = threadIdx.x * V; c < c0; c += blockDim.x * V) {
+      float f[8];
+      if constexpr (sizeof(E) == 2) unpack8(ld_16B(src + c), f);
+      else { const float4 u = *reinterpret_cast<const float4*>(src + c); f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w; }
+#pragma unroll
+      for (int k = 0; k < V; ++k) ss = fmaf(f[k], f[k], ss);
+    }
+  }
+  for (int c = c0 + threadIdx.x; c < n; c += blockDim.x) {
+    const float v = a_to_f(src[c]) + (bs ? bs[c] : 0.f);
+    ss = fmaf(v, v, ss);
+  }
+  return ss;
+}
 
 // One CTA per row; each warp takes heads in turn: q heads -> qbuf (fp32, normed and rotated), key heads and value
 // heads -> the sequence's cache page.
@@ -66,6 +91,17 @@ attn_prep_append_kernel(const E* __restrict__ proj, float* __restrict__ qbuf, E*
   const int pos = e.w + (row - e.y);
   const int page = a.page_table[(size_t)e.x * a.max_pages + pos / a.page_size], off = pos % a.page_size;
   const E* pr = proj + (size_t)row * a.ldp;
+  float r_all[2] = {1.f, 1.f};  // whole: 1 / rms of the row's query and key projections (every CTA of the row forms both)
+  if (a.whole) {
+    __shared__ float red[2][4];
+    float s0 = a.qn ? prep_sum_squares(pr + a.q_off, a.bias ? a.bias + a.q_off : nullptr, a.H * a.D) : 0.f;
+    float s1 = a.kn && !a.q_only ? prep_sum_squares(pr + a.k_off, a.bias ? a.bias + a.k_off : nullptr, a.G * a.D) : 0.f;
+    s0 = warp_sum(s0); s1 = warp_sum(s1);
+    if (lane == 0) { red[0][warp] = s0; red[1][warp] = s1; }
+    __syncthreads();
+    r_all[0] = 1.f / sqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / (a.H * a.D) + a.eps);
+    r_all[1] = 1.f / sqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / (a.G * a.D) + a.eps);
+  }
   // grid.y spreads the heads of a row over CTAs (a decode row would otherwise walk all heads with four warps)
   const int n_items = a.q_only ? a.H : a.H + 2 * a.G;
   for (int item = blockIdx.y * 4 + warp; item < n_items; item += 4 * gridDim.y) {
@@ -76,8 +112,9 @@ attn_prep_append_kernel(const E* __restrict__ proj, float* __restrict__ qbuf, E*
       const E* src = pr + col;
       const float* bs = a.bias ? a.bias + col : nullptr;
       const float* nw = is_q ? a.qn : a.kn;
-      float r = 1.f;
-      if (nw) {
+      float r = r_all[is_q ? 0 : 1];
+      if (nw && a.whole) nw += (size_t)hh * a.D;
+      else if (nw) {
         float ss = 0.f;
         for (int c = lane; c < a.D; c += 32) { const float v = a_to_f(src[c]) + (bs ? bs[c] : 0.f); ss += v * v; }
         ss = warp_sum(ss);
@@ -412,7 +449,7 @@ attn_ragged_merge_kernel(const E* __restrict__ proj, E* __restrict__ out, AttnRu
 // ---- one key/value head shared by all query heads (latent attention over the cached rows, multi-query attention) ----
 // The row-wise kernel above gives every (row, head) its own CTAs, so H heads read the same cached rows H times.  Here a CTA
 // takes HPC heads of a row: a thread loads its key once and forms HPC dot products, and a value load feeds HPC accumulators.
-// Plain causal mask, optional sink, key splits; values in the vector form (4 consecutive dimensions per thread).
+// Causal mask with an optional window, optional sink, key splits; values in the vector form (4 consecutive dimensions per thread).
 __device__ __forceinline__ void load8(const bf16* p, float* f) { unpack8(ld_16B(p), f); }
 __device__ __forceinline__ void load8(const float* p, float* f) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
@@ -436,10 +473,11 @@ attn_shared_kv_kernel(const float* __restrict__ qbuf, const E* __restrict__ kc, 
   const int pos = e.w + (row - e.y);
   const int32_t* pt = a.page_table + (size_t)e.x * a.max_pages;
   for (int i = tid; i < HPC * a.D; i += kAttnThreads) q[i] = qbuf[((size_t)row * a.H + h0) * a.D + i] * a.scale;
-  int jb = 0, je = pos;
+  const int lo = a.window > 0 ? max(pos - a.window + 1, 0) : 0;
+  int jb = lo, je = pos;
   if (a.splits > 1) {
-    const int per = (pos + a.splits) / a.splits;
-    jb = (int)blockIdx.z * per;
+    const int per = (pos - lo + a.splits) / a.splits;
+    jb = lo + (int)blockIdx.z * per;
     je = min(pos, jb + per - 1);
   }
   const int tpg = a.V / 4;                     // threads that cover a value row
@@ -578,9 +616,9 @@ static int launch_shared_kv(const float* qbuf, const void* kc, const void* vc, v
 }
 
 // Does a step of this shape take the shared-key/value kernel, and with how many heads per CTA (0: no)?
-static int shared_kv_heads(int H, int G, int D, int V, int ldv, int chunk, int window, int g_off, const float* cos_v, int dt,
+static int shared_kv_heads(int H, int G, int D, int V, int ldv, int chunk, int first, int g_off, const float* cos_v, int dt,
                            const void* kc, const void* vc, bool plain_only) {
-  if (G != 1 || H < 2 || chunk > 0 || window > 0 || g_off >= 0 || cos_v || plain_only) return 0;
+  if (G != 1 || H < 2 || chunk > 0 || first > 0 || g_off >= 0 || cos_v || plain_only) return 0;
   const size_t es = dt == 0 ? 2 : 4;
   if (D % 8 != 0 || !attn_vec_values(V, ldv) || (ldv * es) % (dt == 0 ? 8 : 16) != 0 || !aligned16(kc) ||
       (reinterpret_cast<uintptr_t>(vc) & 15u) != 0)
@@ -599,11 +637,12 @@ static int shared_kv_heads(int H, int G, int D, int V, int ldv, int chunk, int w
 // key and value sizes are independent; the mask is per row [lo(row), row] with lo from the chunk and the window;
 // the running maximum starts at the sink (in score units) with weight 1; the epilogue turns each output pair back
 // by the row's position and applies the head's gate.  tiles[2t] = entry, tiles[2t+1] = first row of the tile
-// within the entry.
+// within the entry.  PAD: head sizes below the tile's (multiples of 8): the missing columns of keys, values and queries
+// are zeros in shared memory and the missing output columns are not stored.
 constexpr int kRtThreads = 128;
 constexpr int kRtTile = 64;
 
-template <int DK, int DV>
+template <int DK, int DV, bool PAD>
 __global__ void __launch_bounds__(kRtThreads)
 attn_ragged_tc_kernel(const float* __restrict__ qbuf, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
                       const bf16* __restrict__ proj, bf16* __restrict__ out, const int32_t* __restrict__ tiles,
@@ -614,6 +653,7 @@ attn_ragged_tc_kernel(const float* __restrict__ qbuf, const bf16* __restrict__ k
   const uint32_t sQ = smem_u32(smem_tc);
   const uint32_t sK = sQ + kQBytes;
   const uint32_t sV = sK + 2 * kKBytes;
+  const int D = PAD ? a.D : DK, V = PAD ? a.V : DV;  // the heads' own sizes
   pdl_wait();
   pdl_trigger();
   const int h = blockIdx.x, tile_id = gridDim.y - 1 - blockIdx.y;
@@ -629,8 +669,8 @@ attn_ragged_tc_kernel(const float* __restrict__ qbuf, const bf16* __restrict__ k
   for (int id = tid; id < kRtTile * CHK; id += kRtThreads) {
     const int row = id / CHK, c = id - row * CHK;
     uint4 u = make_uint4(0, 0, 0, 0);
-    if (row < n_rows) {
-      const float4* src = reinterpret_cast<const float4*>(qbuf + ((size_t)(e.y + q0 + row) * a.H + h) * DK + c * 8);
+    if (row < n_rows && (!PAD || c * 8 < D)) {
+      const float4* src = reinterpret_cast<const float4*>(qbuf + ((size_t)(e.y + q0 + row) * a.H + h) * D + c * 8);
       const float4 f0 = src[0], f1 = src[1];
       u.x = pack_bf16(f0.x, f0.y); u.y = pack_bf16(f0.z, f0.w); u.z = pack_bf16(f1.x, f1.y); u.w = pack_bf16(f1.z, f1.w);
     }
@@ -646,17 +686,19 @@ attn_ragged_tc_kernel(const float* __restrict__ qbuf, const bf16* __restrict__ k
     // that a pool given as a window of pages is never addressed outside the window
     const int tk = valid ? tok : p_last;
     const size_t rowbase = ((size_t)pt[tk / a.page_size] * a.G + g) * a.page_size + tk % a.page_size;
-    const bf16* ksrc = kc + rowbase * DK;
-    const bf16* vsrc = vc + rowbase * DV;
+    const bf16* ksrc = kc + rowbase * D;
+    const bf16* vsrc = vc + rowbase * V;
 #pragma unroll
     for (int i = 0; i < CHK / 2; ++i) {
       const int c = lhalf * (CHK / 2) + i;
-      cp_async_16B(dK + swz<RBK>(lrow, c), ksrc + c * 8, valid ? 16 : 0);
+      const bool in = !PAD || c * 8 < D;  // a piece outside the row copies nothing (and names an address inside it)
+      cp_async_16B(dK + swz<RBK>(lrow, c), ksrc + (in ? c * 8 : 0), valid && in ? 16 : 0);
     }
 #pragma unroll
     for (int i = 0; i < CHV / 2; ++i) {
       const int c = lhalf * (CHV / 2) + i;
-      cp_async_16B(dV + swz<RBV>(lrow, c), vsrc + c * 8, valid ? 16 : 0);
+      const bool in = !PAD || c * 8 < V;
+      cp_async_16B(dV + swz<RBV>(lrow, c), vsrc + (in ? c * 8 : 0), valid && in ? 16 : 0);
     }
   };
   auto row_lo = [&](int pos) {
@@ -799,14 +841,15 @@ attn_ragged_tc_kernel(const float* __restrict__ qbuf, const bf16* __restrict__ k
       const int pos = qabs[r];
       float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;
       inv *= a.g_chan ? a.oscale : out_gate(proj, a, row, h, 0);
-      bf16* dst = out + row * a.ldo + h * DV + 2 * t4;
-      const bf16* gsrc = a.g_chan ? proj + row * a.ldp + a.g_off + h * DV + 2 * t4 : nullptr;
+      bf16* dst = out + row * a.ldo + h * V + 2 * t4;
+      const bf16* gsrc = a.g_chan ? proj + row * a.ldp + a.g_off + h * V + 2 * t4 : nullptr;
 #pragma unroll
       for (int i = 0; i < DV / 8; ++i) {
+        if (PAD && i * 8 >= V) break;
         float u = o[i][2 * r], v = o[i][2 * r + 1];
         if (a.cos_v) {
           const int pr = i * 4 + t4;  // pair index of columns 8i + 2*t4, +1
-          const float c = a.cos_v[(size_t)pos * (DV / 2) + pr], sn = a.sin_v[(size_t)pos * (DV / 2) + pr];
+          const float c = a.cos_v[(size_t)pos * (V / 2) + pr], sn = a.sin_v[(size_t)pos * (V / 2) + pr];
           const float u2 = u * c + v * sn, v2 = v * c - u * sn;
           u = u2; v = v2;
         }
@@ -820,16 +863,23 @@ attn_ragged_tc_kernel(const float* __restrict__ qbuf, const bf16* __restrict__ k
   }
 }
 
-template <int DK, int DV>
-static int launch_ragged_tc(const float* qbuf, const void* kc, const void* vc, const void* proj, void* out,
+template <int DK, int DV, bool PAD>
+static int launch_ragged_tc_as(const float* qbuf, const void* kc, const void* vc, const void* proj, void* out,
                             const int32_t* tiles, int n_tiles, const AttnRun& a, cudaStream_t s) {
   constexpr int kSmem = kRtTile * DK * 2 + 2 * kRtTile * (DK + DV) * 2;
   static PerDeviceOnce once;
-  DLI_ONCE_PER_DEVICE(once, dev, DLI_CUDA_CALL(cudaFuncSetAttribute(attn_ragged_tc_kernel<DK, DV>,
+  DLI_ONCE_PER_DEVICE(once, dev, DLI_CUDA_CALL(cudaFuncSetAttribute(attn_ragged_tc_kernel<DK, DV, PAD>,
                                                                      cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem)));
-  DLI_LAUNCH("attn_ragged_tc", (attn_ragged_tc_kernel<DK, DV>), dim3(a.H, n_tiles), dim3(kRtThreads), (size_t)kSmem, s,
+  DLI_LAUNCH("attn_ragged_tc", (attn_ragged_tc_kernel<DK, DV, PAD>), dim3(a.H, n_tiles), dim3(kRtThreads), (size_t)kSmem, s,
              qbuf, (const bf16*)kc, (const bf16*)vc, (const bf16*)proj, (bf16*)out, tiles, a);
   return DLI_OK;
+}
+
+template <int DK, int DV>
+static int launch_ragged_tc(const float* qbuf, const void* kc, const void* vc, const void* proj, void* out,
+                            const int32_t* tiles, int n_tiles, const AttnRun& a, cudaStream_t s) {
+  if (a.D == DK && a.V == DV) return launch_ragged_tc_as<DK, DV, false>(qbuf, kc, vc, proj, out, tiles, n_tiles, a, s);
+  return launch_ragged_tc_as<DK, DV, true>(qbuf, kc, vc, proj, out, tiles, n_tiles, a, s);
 }
 
 }  // namespace dli
@@ -842,7 +892,7 @@ int dli_attn_prep_append(const void* proj, float* qbuf, void* k_cache, void* v_c
                          const int32_t* ent, const int32_t* page_table, int max_pages, int page_size, int rows, int H,
                          int G, int D, int V, int rd, int ldp, int q_off, int k_off, int v_off, const float* q_norm,
                          const float* k_norm, float eps, const float* cos_qk, const float* sin_qk, const float* cos_v,
-                         const float* sin_v, int table_len, int dt, const float* bias, int q_only, int halves,
+                         const float* sin_v, int table_len, int dt, const float* bias, int q_only, int halves, int whole_norm,
                          dli_stream_t stream) {
   DLI_CHECK_ARG(proj && qbuf && (q_only || (k_cache && v_cache)) && row_ent && ent && page_table, "dli_attn_prep_append: null pointer");
   DLI_CHECK_ARG(H > 0 && G > 0 && H % G == 0 && D > 0 && V > 0 && D % 2 == 0 && V % 2 == 0 && rd % 2 == 0 && rd <= D,
@@ -851,7 +901,8 @@ int dli_attn_prep_append(const void* proj, float* qbuf, void* k_cache, void* v_c
   DLI_CHECK_ARG(dt == 0 || dt == 1, "element type %d: 0 = bf16, 1 = float", dt);
   if (rows <= 0) return DLI_OK;
   AttnPrep a{row_ent, ent, page_table, max_pages, page_size, H, G, D, V, rd, ldp, q_off, k_off, v_off, q_norm, k_norm,
-             eps, (rd > 0 ? cos_qk : nullptr), sin_qk, cos_v, sin_v, table_len, bias, q_only ? 1 : 0, halves ? 1 : 0};
+             eps, (rd > 0 ? cos_qk : nullptr), sin_qk, cos_v, sin_v, table_len, bias, q_only ? 1 : 0, halves ? 1 : 0,
+             whole_norm && (q_norm || k_norm) ? 1 : 0};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int items = q_only ? H : H + 2 * G;
   const dim3 pgrid(rows, rows <= 64 ? (items + 3) / 4 : 1);
@@ -884,7 +935,7 @@ int dli_attn_ragged(const float* qbuf, const void* k_cache, const void* v_cache,
   const size_t smem = sizeof(float) * (D + kAttnThreads + 8 + (size_t)groups * V);
   DLI_CHECK_ARG(smem <= 48 * 1024, "dli_attn_ragged: key size %d needs %zu bytes of shared memory", D, smem);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  const int hpc = shared_kv_heads(H, G, D, V, ldv ? ldv : V, chunk, window, g_off, cos_v, dt, k_cache, v_cache,
+  const int hpc = shared_kv_heads(H, G, D, V, ldv ? ldv : V, chunk, first, g_off, cos_v, dt, k_cache, v_cache,
                                   r1 != nullptr || cap > 0.f || out_scale != 1.f || a.ldo != H * V);
   if (hpc) {
     int rc;
@@ -904,8 +955,8 @@ int dli_attn_ragged(const float* qbuf, const void* k_cache, const void* v_cache,
 }
 
 int dli_attn_ragged_tc_supported(int D, int V, int dt) {
-  return dt == 0 && ((D == 64 && V == 64) || (D == 128 && V == 128) || (D == 64 && V == 128) || (D == 128 && V == 64) ||
-                     (D == 128 && V == 256));
+  // tiles of 64 / 128 key and 64 / 128 / 256 value columns; smaller heads leave a part of the next larger tile empty
+  return dt == 0 && D % 8 == 0 && V % 8 == 0 && D >= 32 && V >= 32 && D <= 128 && V <= 256;
 }
 
 int dli_attn_ragged_tc(const float* qbuf, const void* k_cache, const void* v_cache, const void* proj, void* out,
@@ -925,10 +976,10 @@ int dli_attn_ragged_tc(const float* qbuf, const void* k_cache, const void* v_cac
   AttnRun a{nullptr, ent, page_table, max_pages, page_size, H, G, D, V, scale, chunk, window, first, sink, ldp, g_off, cos_v, sin_v, V, 1, nullptr, r1, r2,
             cap > 0.f ? cap : 0.f, g_off >= 0 && g_chan ? 1 : 0, out_scale, ldo ? ldo : H * V};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (D == 64 && V == 64) return launch_ragged_tc<64, 64>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);
-  if (D == 128 && V == 128) return launch_ragged_tc<128, 128>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);
-  if (D == 64 && V == 128) return launch_ragged_tc<64, 128>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);
-  if (D == 128 && V == 64) return launch_ragged_tc<128, 64>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);
+  if (D <= 64 && V <= 64) return launch_ragged_tc<64, 64>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);
+  if (D <= 64 && V <= 128) return launch_ragged_tc<64, 128>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);
+  if (V <= 64) return launch_ragged_tc<128, 64>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);
+  if (V <= 128) return launch_ragged_tc<128, 128>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);
   return launch_ragged_tc<128, 256>(qbuf, k_cache, v_cache, proj, out, tiles, n_tiles, a, s);
 }
 

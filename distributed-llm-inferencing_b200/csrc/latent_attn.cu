@@ -9,7 +9,8 @@
 // (dli_attn_ragged with ldv = K + R):
 //   dli_latent_prep      c_q = rmsnorm(W_dq h) -> operand of the query up-projection; c, rotated k_r -> the pool
 //   dli_latent_q_absorb  q~[h] = [U_k[h]^T q_n[h] | rot(q_r[h])] -> fp32 query rows of size K + R
-//   dli_latent_v_up      out[h] = (U_v[h] o~[h]) * sigmoid(gate[h])   with o~ the attention output in the latent
+//   dli_latent_v_up      out[h] = (U_v[h] o~[h]) * sigmoid(gate[h])   with o~ the attention output in the latent; the gate
+//                        has a column per output channel or (g_head) one per head
 // Rotation: from a host-made fp32 cos/sin table [positions, R/2]; pair i is entries (2i, 2i+1) (`halves` == 0,
 // interleaved) or entries (i, i + R/2) (`halves` != 0).  A model without a query latent (Q == 0) projects its
 // queries directly and skips that part of dli_latent_prep.  Norms, rotation and the absorbed queries are fp32; E
@@ -151,12 +152,13 @@ latent_q_absorb_kernel(const E* __restrict__ q, const E* __restrict__ uk, float*
   }
 }
 
-// out[row, h*V + v] = (sum_k uv[h, v, k] * o[row, h, k]) * sigmoid(proj[row, g_off + h*V + v])   (g_off < 0: no gate)
+// out[row, h*V + v] = (sum_k uv[h, v, k] * o[row, h, k]) * sigmoid(proj[row, g_off + h*V + v])   (g_off < 0: no gate; g_head:
+// one gate column per head, g_off + h)
 // Grid (row tiles, heads); one warp per output v, lanes across K, the tile's latent outputs in shared memory.
 template <typename E>
 __global__ void __launch_bounds__(256)
 latent_v_up_kernel(const E* __restrict__ o, const E* __restrict__ uv, const E* __restrict__ proj, E* __restrict__ out,
-                   int rows, int H, int V, int K, int ldp, int g_off) {
+                   int rows, int H, int V, int K, int ldp, int g_off, int g_head) {
   extern __shared__ float os[];  // [kLatRows][Kp], Kp = K rounded up to 256
   pdl_wait();
   pdl_trigger();
@@ -201,7 +203,7 @@ latent_v_up_kernel(const E* __restrict__ o, const E* __restrict__ uv, const E* _
 #pragma unroll
       for (int r = 0; r < kLatRows; ++r) if (r == lane) val = acc[r];
       const size_t row = r0 + lane;
-      if (g_off >= 0) val *= 1.f / (1.f + expf(-l_to_f(proj[row * ldp + g_off + h * V + v])));
+      if (g_off >= 0) val *= 1.f / (1.f + expf(-l_to_f(proj[row * ldp + g_off + (g_head ? h : h * V + v)])));
       out[(row * H + h) * V + v] = l_from_f<E>(val);
     }
   }
@@ -288,7 +290,7 @@ int dli_latent_q_absorb(const void* q, const void* uk, float* qbuf, const int32_
 }
 
 int dli_latent_v_up(const void* o, const void* uv, const void* proj, void* out, int rows, int H, int V, int K, int ldp,
-                    int g_off, int dt, dli_stream_t stream) {
+                    int g_off, int g_head, int dt, dli_stream_t stream) {
   DLI_CHECK_ARG(o && uv && out && (g_off < 0 || proj), "dli_latent_v_up: null pointer");
   DLI_CHECK_ARG(H > 0 && V > 0 && K > 0 && (size_t)kLatRows * ((K + 255) / 256 * 256) * sizeof(float) <= 48 * 1024,
                 "dli_latent_v_up: H=%d V=%d K=%d (K <= %d)", H, V, K, 48 * 1024 / (kLatRows * 4));
@@ -297,8 +299,8 @@ int dli_latent_v_up(const void* o, const void* uv, const void* proj, void* out, 
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const dim3 grid((rows + kLatRows - 1) / kLatRows, H, rows <= 16 ? (V + 31) / 32 : 1);
   const size_t smem = (size_t)kLatRows * ((K + 255) / 256 * 256) * sizeof(float);
-  if (dt == 0) DLI_LAUNCH("latent_v_up", latent_v_up_kernel<bf16>, grid, dim3(256), smem, s, (const bf16*)o, (const bf16*)uv, (const bf16*)proj, (bf16*)out, rows, H, V, K, ldp, g_off);
-  else DLI_LAUNCH("latent_v_up", latent_v_up_kernel<float>, grid, dim3(256), smem, s, (const float*)o, (const float*)uv, (const float*)proj, (float*)out, rows, H, V, K, ldp, g_off);
+  if (dt == 0) DLI_LAUNCH("latent_v_up", latent_v_up_kernel<bf16>, grid, dim3(256), smem, s, (const bf16*)o, (const bf16*)uv, (const bf16*)proj, (bf16*)out, rows, H, V, K, ldp, g_off, g_head ? 1 : 0);
+  else DLI_LAUNCH("latent_v_up", latent_v_up_kernel<float>, grid, dim3(256), smem, s, (const float*)o, (const float*)uv, (const float*)proj, (float*)out, rows, H, V, K, ldp, g_off, g_head ? 1 : 0);
   return DLI_OK;
 }
 

@@ -5,14 +5,17 @@
 //                   without renormalisation, s itself, in both cases times `wscale`.  With groups > 1 the outputs form
 //                   that many equal groups of neighbours, a group's score is its largest s + correction, and only
 //                   outputs of the `keep` best groups can be chosen.
+//                   Scores may be a sigmoid of each logit instead of the softmax (score == 1).  One more router row (sg_w)
+//                   gives the shared expert's weight, its sigmoid, in sg[row].
 //                   The last n_identity router outputs are experts that return their input: their weights are
 //                   summed into idw[row].  Written: the dense weight row wts[row, 0 .. n_real) (0 for experts that
 //                   were not chosen), idw[row], and the choice itself (sel_idx / sel_w [row, top]).
 //   dli_moe_act     the experts' activation on the stacked gate/up projection of all experts:
 //                   g = min(g, limit), u = clamp(u, -limit, limit), a = g * sigmoid(alpha g) * (u + 1), times the
 //                   expert's routing weight, so that ONE down projection over the concatenated experts is the
-//                   weighted sum of their outputs.  A shared expert (its own size and limit, weight 1) is the last
-//                   block.  mode 1: experts without a gate, a = max(u, 0)^2 on the stacked up projections.
+//                   weighted sum of their outputs.  A shared expert (its own size and limit, weight 1 or sg[row]) is the
+//                   last block.  w_in: the weight scales the expert's INPUT instead (its projections have no biases, so
+//                   that is a factor on g and u in front of the activation).  mode 1: experts without a gate, a = max(u, 0)^2 on the stacked up projections.
 //                   mode 2: a = silu(g) * u, no limits.
 #include <math.h>
 
@@ -31,7 +34,7 @@ template <> __device__ __forceinline__ bf16 x_from_f<bf16>(float v) { return __f
 // One CTA per row: a warp per router output for the logits, then one warp does the softmax and the choice (moe_route.cuh).
 __global__ void __launch_bounds__(512)
 moe_route_kernel(const float* __restrict__ h, int d, RouteArgs ra) {
-  extern __shared__ float zs[];  // [n_out] scores, [n_out] choice scores, [groups] group scores
+  extern __shared__ float zs[];  // moe_route_floats(n_out, groups)
   pdl_wait();
   pdl_trigger();
   moe_route_row(h + (size_t)blockIdx.x * d, d, blockIdx.x, ra, zs);
@@ -46,6 +49,8 @@ struct MoeAct {
   int ld;                   // row stride of gu
   int mode;                 // 0: clamped gated form; 1: no gate, max(u, 0)^2, columns [e*ff, +ff) of gu (shared: after them); 2: silu(g) * u
   int vec;                  // modes 1 and 2: sizes and pointers allow 16-byte accesses
+  int w_in;                 // 1: the routing weight scales the expert's input (g and u), 0: its output
+  const float* sg;          // [rows] or NULL: weight of the shared expert's output
 };
 
 // one gated activation, modes 0 and 2
@@ -54,6 +59,14 @@ __device__ __forceinline__ float moe_gated(float g, float u, float lim, const Mo
   g = fminf(g, lim);
   u = fminf(fmaxf(u, -lim), lim);
   return g / (1.f + expf(-a.alpha * g)) * (u + 1.f);
+}
+// with the routing weight where it belongs: wi on the input, wo on the output (one of them is 1)
+__device__ __forceinline__ float moe_gated_w(float g, float u, float lim, float wi, float wo, const MoeAct& a) {
+  return moe_gated(g * wi, u * wi, lim, a) * wo;
+}
+__device__ __forceinline__ float moe_relu2_w(float u, float wi, float wo) {
+  const float r = fmaxf(u * wi, 0.f);
+  return r * r * wo;
 }
 
 // act[row, e*ff + f] and act[row, n_exp*ff + f] (shared); a row's channels go to one CTA, or to several for few rows.
@@ -66,11 +79,14 @@ moe_act_kernel(const E* __restrict__ gu, const float* __restrict__ wts, E* __res
   const E* g = gu + row * a.ld;
   const int F = a.n_exp * a.ff + a.ff_s;
   E* out = act + row * F;
+  const float sgw = a.sg && a.ff_s ? a.sg[row] : 1.f;
   if (a.mode == 1 && a.vec) {
     // experts without a gate, 16 bytes per thread and access: the V elements lie in one expert (ff, ff_s multiples of V)
     constexpr int V = 16 / (int)sizeof(E);
     for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * V; i < F; i += blockDim.x * gridDim.y * V) {
-      const float wt = i < a.n_exp * a.ff ? wts[row * a.n_exp + i / a.ff] : 1.f;
+      const bool routed = i < a.n_exp * a.ff;
+      const float wt = routed ? wts[row * a.n_exp + i / a.ff] : sgw;
+      const float wi = routed && a.w_in ? wt : 1.f, wo = routed && a.w_in ? 1.f : wt;
       uint4 o = make_uint4(0, 0, 0, 0);
       if (wt != 0.f) {
         const uint4 u = *reinterpret_cast<const uint4*>(g + i);
@@ -78,13 +94,13 @@ moe_act_kernel(const E* __restrict__ gu, const float* __restrict__ wts, E* __res
           float f[8];
           unpack8(u, f);
 #pragma unroll
-          for (int k = 0; k < 8; ++k) { const float r = fmaxf(f[k], 0.f); f[k] = r * r * wt; }
+          for (int k = 0; k < 8; ++k) f[k] = moe_relu2_w(f[k], wi, wo);
           o = pack8(f);
         } else {
           const float f[4] = {__uint_as_float(u.x), __uint_as_float(u.y), __uint_as_float(u.z), __uint_as_float(u.w)};
           float r[4];
 #pragma unroll
-          for (int k = 0; k < 4; ++k) { const float t = fmaxf(f[k], 0.f); r[k] = t * t * wt; }
+          for (int k = 0; k < 4; ++k) r[k] = moe_relu2_w(f[k], wi, wo);
           o = make_uint4(__float_as_uint(r[0]), __float_as_uint(r[1]), __float_as_uint(r[2]), __float_as_uint(r[3]));
         }
       }
@@ -98,7 +114,8 @@ moe_act_kernel(const E* __restrict__ gu, const float* __restrict__ wts, E* __res
     for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * V; i < F; i += blockDim.x * gridDim.y * V) {
       const bool routed = i < a.n_exp * a.ff;
       const int e = routed ? i / a.ff : a.n_exp, f = i - e * a.ff, ff = routed ? a.ff : a.ff_s;
-      const float wt = routed ? wts[row * a.n_exp + e] : 1.f;
+      const float wt = routed ? wts[row * a.n_exp + e] : sgw;
+      const float wi = routed && a.w_in ? wt : 1.f, wo = routed && a.w_in ? 1.f : wt;
       uint4 o = make_uint4(0, 0, 0, 0);
       if (wt != 0.f) {
         const E* gp = g + (size_t)e * 2 * a.ff + f;
@@ -108,13 +125,13 @@ moe_act_kernel(const E* __restrict__ gu, const float* __restrict__ wts, E* __res
           unpack8(gu4, gf);
           unpack8(uu4, uf);
 #pragma unroll
-          for (int k = 0; k < 8; ++k) gf[k] = moe_gated(gf[k], uf[k], 0.f, a) * wt;
+          for (int k = 0; k < 8; ++k) gf[k] = moe_gated_w(gf[k], uf[k], 0.f, wi, wo, a);
           o = pack8(gf);
         } else {
-          o.x = __float_as_uint(moe_gated(__uint_as_float(gu4.x), __uint_as_float(uu4.x), 0.f, a) * wt);
-          o.y = __float_as_uint(moe_gated(__uint_as_float(gu4.y), __uint_as_float(uu4.y), 0.f, a) * wt);
-          o.z = __float_as_uint(moe_gated(__uint_as_float(gu4.z), __uint_as_float(uu4.z), 0.f, a) * wt);
-          o.w = __float_as_uint(moe_gated(__uint_as_float(gu4.w), __uint_as_float(uu4.w), 0.f, a) * wt);
+          o.x = __float_as_uint(moe_gated_w(__uint_as_float(gu4.x), __uint_as_float(uu4.x), 0.f, wi, wo, a));
+          o.y = __float_as_uint(moe_gated_w(__uint_as_float(gu4.y), __uint_as_float(uu4.y), 0.f, wi, wo, a));
+          o.z = __float_as_uint(moe_gated_w(__uint_as_float(gu4.z), __uint_as_float(uu4.z), 0.f, wi, wo, a));
+          o.w = __float_as_uint(moe_gated_w(__uint_as_float(gu4.w), __uint_as_float(uu4.w), 0.f, wi, wo, a));
         }
       }
       *reinterpret_cast<uint4*>(out + i) = o;
@@ -123,17 +140,18 @@ moe_act_kernel(const E* __restrict__ gu, const float* __restrict__ wts, E* __res
   }
   for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < F; i += blockDim.x * gridDim.y) {
     float gv, uv, lim, wt;
+    const bool routed = i < a.n_exp * a.ff;
     if (a.mode == 1) {
-      wt = 1.f;
-      if (i < a.n_exp * a.ff) {
+      wt = sgw;
+      if (routed) {
         wt = wts[row * a.n_exp + i / a.ff];
         if (wt == 0.f) { out[i] = x_from_f<E>(0.f); continue; }
       }
-      const float u = fmaxf(x_to_f(g[i]), 0.f);
-      out[i] = x_from_f<E>(u * u * wt);
+      const bool in = routed && a.w_in;
+      out[i] = x_from_f<E>(moe_relu2_w(x_to_f(g[i]), in ? wt : 1.f, in ? 1.f : wt));
       continue;
     }
-    if (i < a.n_exp * a.ff) {
+    if (routed) {
       const int e = i / a.ff, f = i - e * a.ff;
       wt = wts[row * a.n_exp + e];
       if (wt == 0.f) { out[i] = x_from_f<E>(0.f); continue; }
@@ -142,12 +160,13 @@ moe_act_kernel(const E* __restrict__ gu, const float* __restrict__ wts, E* __res
       lim = a.limit;
     } else {
       const int f = i - a.n_exp * a.ff;
-      wt = 1.f;
+      wt = sgw;
       gv = x_to_f(g[(size_t)a.n_exp * 2 * a.ff + f]);
       uv = x_to_f(g[(size_t)a.n_exp * 2 * a.ff + a.ff_s + f]);
       lim = a.limit_s;
     }
-    out[i] = x_from_f<E>(moe_gated(gv, uv, lim, a) * wt);
+    const bool in = routed && a.w_in;
+    out[i] = x_from_f<E>(moe_gated_w(gv, uv, lim, in ? wt : 1.f, in ? 1.f : wt, a));
   }
 }
 
@@ -188,7 +207,9 @@ moe_sel_act_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w_gu, co
   }
   for (int c = threadIdx.x; c < d; c += blockDim.x) xs[c] = __bfloat162float(x[(size_t)row * d + c]);
   __syncthreads();
-  const float wt = shared ? 1.f : sel_w[row * top + k];
+  const float wt = shared ? (a.sg ? a.sg[row] : 1.f) : sel_w[row * top + k];
+  const bool in = !shared && a.w_in;
+  const float wi = in ? wt : 1.f, wo = in ? 1.f : wt;
   const float lim = shared ? a.limit_s : a.limit;
   if (a.mode == 1) {
     // experts without a gate: one weight row per output, two outputs at a time
@@ -213,8 +234,8 @@ moe_sel_act_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w_gu, co
       u0 = warp_sum(u0); u1 = warp_sum(u1);
       if (lane < 2 && f + lane < ff) {
         float u = lane ? u1 : u0;
-        u = fmaxf(__bfloat162float(__float2bfloat16_rn(u)), 0.f);  // the projection's output is a bf16 row, as on the dense path
-        out[f + lane] = __float2bfloat16_rn(u * u * wt);
+        u = __bfloat162float(__float2bfloat16_rn(u));  // the projection's output is a bf16 row, as on the dense path
+        out[f + lane] = __float2bfloat16_rn(moe_relu2_w(u, wi, wo));
       }
     }
     return;
@@ -250,7 +271,7 @@ moe_sel_act_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w_gu, co
       float g = lane ? g1 : g0, u = lane ? u1 : u0;
       g = __bfloat162float(__float2bfloat16_rn(g));  // the projection's output is a bf16 row, as on the dense path
       u = __bfloat162float(__float2bfloat16_rn(u));
-      out[f + lane] = __float2bfloat16_rn(moe_gated(g, u, lim, a) * wt);
+      out[f + lane] = __float2bfloat16_rn(moe_gated_w(g, u, lim, wi, wo, a));
     }
   }
 }
@@ -303,22 +324,23 @@ extern "C" {
 
 int dli_moe_route(const float* h, const float* w_router, const float* correction, float* wts, float* idw, int32_t* sel_idx,
                   float* sel_w, int rows, int d, int n_out, int n_real, int top, int groups, int keep, float wscale,
-                  int renorm, const float* logit_bias, dli_stream_t stream) {
-  DLI_CHECK_ARG(h && w_router && wts && idw && sel_idx && sel_w, "dli_moe_route: null pointer");
+                  int renorm, const float* logit_bias, int score, const float* sg_w, float* sg, dli_stream_t stream) {
+  DLI_CHECK_ARG(h && w_router && wts && idw && sel_idx && sel_w && (!sg_w || sg), "dli_moe_route: null pointer");
+  DLI_CHECK_ARG(score == 0 || score == 1, "dli_moe_route: score %d: 0 = softmax, 1 = sigmoid", score);
   if (groups < 1) groups = 1;
   DLI_CHECK_ARG(groups == 1 || (n_out % groups == 0 && keep >= 1 && keep <= groups && keep * (n_out / groups) >= top),
                 "dli_moe_route: %d router outputs in %d groups of which %d are kept, top %d", n_out, groups, keep, top);
   DLI_CHECK_ARG(d > 0 && n_out > 0 && n_real >= 0 && n_real <= n_out && top > 0 && top <= n_out && n_out <= 4096,
                 "dli_moe_route: %d router outputs (%d real experts), top %d", n_out, n_real, top);
   if (rows <= 0) return DLI_OK;
-  RouteArgs ra{w_router, correction, wts, idw, sel_idx, sel_w, n_out, n_real, top, groups, keep, wscale, renorm, logit_bias};
-  DLI_LAUNCH("moe_route", moe_route_kernel, dim3(rows), dim3(rows <= 64 ? 512 : 256), (size_t)(2 * n_out + groups) * sizeof(float),
+  RouteArgs ra{w_router, correction, wts, idw, sel_idx, sel_w, n_out, n_real, top, groups, keep, wscale, renorm, logit_bias, score, sg_w, sg};
+  DLI_LAUNCH("moe_route", moe_route_kernel, dim3(rows), dim3(rows <= 64 ? 512 : 256), (size_t)moe_route_floats(n_out, groups) * sizeof(float),
              static_cast<cudaStream_t>(stream), h, d, ra);
   return DLI_OK;
 }
 
 int dli_moe_act(const void* gu, const float* wts, void* act, int rows, int n_exp, int ff, float limit, int ff_s,
-                float limit_s, float alpha, int ld, int dt, int mode, dli_stream_t stream) {
+                float limit_s, float alpha, int ld, int dt, int mode, int w_in, const float* sg, dli_stream_t stream) {
   DLI_CHECK_ARG(gu && act && (wts || n_exp == 0) && n_exp >= 0 && ff >= 0 && ff_s >= 0 && n_exp * ff + ff_s > 0 &&
                     mode >= 0 && mode <= 2 && ld >= (mode == 1 ? 1 : 2) * (n_exp * ff + ff_s),
                 "dli_moe_act: null pointer or bad shape");
@@ -326,7 +348,7 @@ int dli_moe_act(const void* gu, const float* wts, void* act, int rows, int n_exp
   if (rows <= 0) return DLI_OK;
   const int per = dt == 0 ? 8 : 4;
   const int vec = mode >= 1 && ff % per == 0 && ff_s % per == 0 && ld % per == 0 && aligned16(gu) && aligned16(act);
-  MoeAct a{n_exp, ff, limit, ff_s, limit_s, alpha, ld, mode, vec};
+  MoeAct a{n_exp, ff, limit, ff_s, limit_s, alpha, ld, mode, vec, w_in ? 1 : 0, sg};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   const int work = (n_exp * ff + ff_s) / (vec ? per : 1);
   const int gy = rows <= 64 ? min(64, (work + 255) / 256) : (work >= 4096 ? 4 : 1);  // few rows, or long rows: several CTAs per row
@@ -341,12 +363,12 @@ int dli_moe_sel_supported(int d, int ff, int ff_s, int top) {
 
 int dli_moe_sel_bf16(const void* x, const void* w_gu, const void* w_down, const int32_t* sel_idx, const float* sel_w,
                      void* act_sel, void* y, int rows, int d, int n_exp, int top, int ff, float limit, int ff_s,
-                     float limit_s, float alpha, int mode, dli_stream_t stream) {
+                     float limit_s, float alpha, int mode, int w_in, const float* sg, dli_stream_t stream) {
   DLI_CHECK_ARG(x && w_gu && w_down && sel_idx && sel_w && act_sel && y && mode >= 0 && mode <= 2, "dli_moe_sel_bf16: null pointer");
   DLI_CHECK_ARG(n_exp >= 0 && top >= 0 && dli_moe_sel_supported(d, ff, ff_s, top) && aligned16(w_gu) && aligned16(w_down),
                 "dli_moe_sel_bf16: sizes d=%d ff=%d ff_s=%d must be multiples of 8 and fit shared memory", d, ff, ff_s);
   if (rows <= 0) return DLI_OK;
-  MoeAct a{n_exp, ff, limit, ff_s, limit_s, alpha, 0, mode, 0};
+  MoeAct a{n_exp, ff, limit, ff_s, limit_s, alpha, 0, mode, 0, w_in ? 1 : 0, sg};
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   static PerDeviceOnce once_a, once_d;
   DLI_ONCE_PER_DEVICE(once_a, dev, DLI_CUDA_CALL(cudaFuncSetAttribute(moe_sel_act_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024)));

@@ -1,7 +1,8 @@
 // The router of a mixture of experts for ONE row, shared by dli_moe_route and by kernels that have the router's input row at
-// hand (the closing kernel of pre-norm layers).  Every thread of the CTA calls it; zs is shared scratch of
-// 2 * n_out + groups floats.  Logits in fp32, a warp per router output; then one warp does the softmax, the groups and
-// the choice.  Nothing after the call may need all threads: the warps other than the first return early.
+// hand (the closing kernels of pre-norm layers).  Every thread of the CTA calls moe_route_row; zs is shared scratch of
+// moe_route_floats(n_out, groups) floats.  Logits in fp32, a warp per router output; then one warp does the scores, the
+// groups and the choice (moe_route_choose, which kernels that form the logits of several rows themselves call directly).
+// Nothing after the call may need all threads: the warps other than the first return early.
 #pragma once
 #include <math.h>
 
@@ -21,11 +22,34 @@ struct RouteArgs {
   float wscale;
   int renorm;             // 1: weights divided by the sum of the chosen scores (the softmax over the chosen logits alone)
   const float* zb;        // [n_out] or NULL: added to the logits
+  int score;              // scores of the logits: 0 = softmax over all outputs, 1 = a sigmoid of each
+  const float* sg_w;      // [d] or NULL: one more row of the router, whose sigmoid is the shared expert's weight ...
+  float* sg;              // ... [rows]
 };
 
-// hr may have been written earlier in the same kernel (no __restrict__: plain coherent loads).
-__device__ __forceinline__ void moe_route_row(const float* hr, int d, size_t row, const RouteArgs& ra, float* zs) {
-  const float* __restrict__ wr = ra.wr;
+// logits and scores [n_out], choice scores [n_out], group scores [groups], the shared expert's logit
+__host__ __device__ inline int moe_route_floats(int n_out, int groups) { return 2 * n_out + groups + 1; }
+
+// row . w over d channels by one warp (every lane gets the sum); hr may have been written earlier in the same kernel
+__device__ __forceinline__ float moe_route_dot(const float* hr, const float* __restrict__ w, int d, int lane) {
+  float acc = 0.f;
+  if ((d & 3) == 0) {  // 16-byte loads, four in flight per lane
+    const float4* h4 = reinterpret_cast<const float4*>(hr);
+    const float4* w4 = reinterpret_cast<const float4*>(w);
+#pragma unroll 4
+    for (int c = lane; c < d / 4; c += 32) {
+      const float4 a = h4[c], b = w4[c];
+      acc = fmaf(a.x, b.x, acc); acc = fmaf(a.y, b.y, acc); acc = fmaf(a.z, b.z, acc); acc = fmaf(a.w, b.w, acc);
+    }
+  } else {
+    for (int c = lane; c < d; c += 32) acc = fmaf(hr[c], w[c], acc);
+  }
+  return warp_sum(acc);
+}
+
+// Scores, groups and choice of one row by one warp from its logits in zs (with the shared expert's logit behind the group
+// scores).
+__device__ __forceinline__ void moe_route_choose(size_t row, const RouteArgs& ra, float* zs) {
   const float* __restrict__ corr = ra.corr;
   float* __restrict__ wts = ra.wts;
   float* __restrict__ idw = ra.idw;
@@ -35,37 +59,28 @@ __device__ __forceinline__ void moe_route_row(const float* hr, int d, size_t row
   const float wscale = ra.wscale;
   float* cs = zs + n_out;
   float* gm = cs + n_out;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  for (int o = warp; o < n_out; o += nw) {
-    const float* w = wr + (size_t)o * d;
-    float acc = 0.f;
-    if ((d & 3) == 0) {  // 16-byte loads, four in flight per lane
-      const float4* h4 = reinterpret_cast<const float4*>(hr);
-      const float4* w4 = reinterpret_cast<const float4*>(w);
-#pragma unroll 4
-      for (int c = lane; c < d / 4; c += 32) {
-        const float4 a = h4[c], b = w4[c];
-        acc = fmaf(a.x, b.x, acc); acc = fmaf(a.y, b.y, acc); acc = fmaf(a.z, b.z, acc); acc = fmaf(a.w, b.w, acc);
-      }
-    } else {
-      for (int c = lane; c < d; c += 32) acc = fmaf(hr[c], w[c], acc);
+  const int lane = threadIdx.x & 31;
+  if (ra.sg_w && lane == 0) ra.sg[row] = 1.f / (1.f + expf(-gm[groups]));
+  if (ra.score == 1) {
+    for (int o = lane; o < n_out; o += 32) {
+      const float z = zs[o], s = 1.f / (1.f + expf(-z));
+      zs[o] = s;
+      cs[o] = corr ? s + corr[o] : z;  // without a correction the logit orders alike, also where fp32's sigmoid is already 1
+      if (o < n_real) wts[row * n_real + o] = 0.f;
     }
-    acc = warp_sum(acc);
-    if (lane == 0) zs[o] = acc + (ra.zb ? ra.zb[o] : 0.f);
-  }
-  __syncthreads();
-  if (warp != 0) return;
-  float mx = -INFINITY;
-  for (int o = lane; o < n_out; o += 32) mx = fmaxf(mx, zs[o]);
-  mx = warp_max(mx);
-  float sum = 0.f;
-  for (int o = lane; o < n_out; o += 32) sum += expf(zs[o] - mx);
-  sum = warp_sum(sum);
-  for (int o = lane; o < n_out; o += 32) {
-    const float s = expf(zs[o] - mx) / sum;
-    zs[o] = s;
-    cs[o] = s + (corr ? corr[o] : 0.f);
-    if (o < n_real) wts[row * n_real + o] = 0.f;
+  } else {
+    float mx = -INFINITY;
+    for (int o = lane; o < n_out; o += 32) mx = fmaxf(mx, zs[o]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int o = lane; o < n_out; o += 32) sum += expf(zs[o] - mx);
+    sum = warp_sum(sum);
+    for (int o = lane; o < n_out; o += 32) {
+      const float s = expf(zs[o] - mx) / sum;
+      zs[o] = s;
+      cs[o] = s + (corr ? corr[o] : 0.f);
+      if (o < n_real) wts[row * n_real + o] = 0.f;
+    }
   }
   __syncwarp();
   if (groups > 1) {
@@ -130,6 +145,23 @@ __device__ __forceinline__ void moe_route_row(const float* hr, int d, size_t row
     }
     idw[row] = ident;
   }
+}
+
+// hr may have been written earlier in the same kernel (no __restrict__: plain coherent loads).
+__device__ __forceinline__ void moe_route_row(const float* hr, int d, size_t row, const RouteArgs& ra, float* zs) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const int n_log = ra.n_out + (ra.sg_w ? 1 : 0);
+  for (int o = warp; o < n_log; o += nw) {
+    const bool own = o < ra.n_out;
+    const float z = moe_route_dot(hr, own ? ra.wr + (size_t)o * d : ra.sg_w, d, lane);
+    if (lane == 0) {
+      if (own) zs[o] = z + (ra.zb ? ra.zb[o] : 0.f);
+      else zs[2 * ra.n_out + ra.groups] = z;
+    }
+  }
+  __syncthreads();
+  if (warp != 0) return;
+  moe_route_choose(row, ra, zs);
 }
 
 }  // namespace dli

@@ -168,7 +168,7 @@ layer_close_kernel(const E* __restrict__ y, float* __restrict__ x, E* __restrict
     if (out_e) st_e<VEC>(out_e + o + c, h);
   }
   if (a.has_route) {
-    extern __shared__ float route_scratch[];  // 2 * n_out + groups floats
+    extern __shared__ float route_scratch[];  // moe_route_floats(n_out, groups)
     __syncthreads();                          // the row of out_f is complete
     moe_route_row(a.out_f + o, d, row, a.route, route_scratch);
   }
@@ -231,7 +231,7 @@ int dli_layer_close(const void* y, const float* bias, const float* idw, const fl
   if (rows <= 0) return DLI_OK;
   LayerClose a{bias, idw, h_in, ls, xs, xs_stride, n_prev, dwa, w_next, shift, tail, ent, out_f, eps, d, w_router ? 1 : 0,
                RouteArgs{w_router, correction, r_wts, r_idw, r_sel_idx, r_sel_w, n_out, n_real, top, groups, keep, wscale, renorm, logit_bias}};
-  const size_t smem = w_router ? (size_t)(2 * n_out + groups) * sizeof(float) : 0;
+  const size_t smem = w_router ? (size_t)moe_route_floats(n_out, groups) * sizeof(float) : 0;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   // 16-byte accesses when every row and vector starts on such a boundary
   auto al = [](const void* p, uintptr_t n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; };

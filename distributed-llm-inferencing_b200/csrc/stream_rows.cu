@@ -172,7 +172,7 @@ int dli_streams_close(const void* y, float* x, size_t xs_stride, int n_streams, 
                               (groups == 1 || (n_out % groups == 0 && keep >= 1 && keep <= groups && keep * (n_out / groups) >= top))),
                 "dli_streams_close: the router needs the norm and its outputs; %d outputs (%d real), top %d, %d groups of which %d are kept",
                 n_out, n_real, top, groups, keep);
-  const size_t smem = sizeof(float) * ((w_next ? ((size_t)d + 3) / 4 * 4 : 0) + (w_router ? (size_t)2 * n_out + groups : 0));
+  const size_t smem = sizeof(float) * ((w_next ? ((size_t)d + 3) / 4 * 4 : 0) + (w_router ? (size_t)moe_route_floats(n_out, groups) : 0));
   DLI_CHECK_ARG(smem <= 48 * 1024, "dli_streams_close: width %d needs %zu bytes of shared memory", d, smem);
   if (rows <= 0) return DLI_OK;
   StreamsClose a{x, xs_stride, mix, outw, in_next, w_next, out_f, eps, d, w_router ? 1 : 0,

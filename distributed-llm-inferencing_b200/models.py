@@ -1,9 +1,9 @@
 """Model registry: which engine serves a model directory.
 
 config.json decides: `model_type` llama / mistral / gpt2 -> engine.ShardEngine (uniform stacks, Hugging Face tensor
-names); `architecture` Sokevik, Togalorn, Fubepel, Gimudra or Salizen -> ragged_engine.RaggedEngine with the layer list that
-sokevik.py / togalorn.py / fubepel.py / gimudra.py / salizen.py read from the configuration.  The worker, the trace replayer (bin/trace_run) and bench.py all come
-through here.
+names); `architecture` Sokevik, Togalorn, Fubepel, Gimudra, Salizen or Finezen -> ragged_engine.RaggedEngine with the layer
+list that sokevik.py / togalorn.py / fubepel.py / gimudra.py / salizen.py / finezen.py read from the configuration.  The worker,
+the trace replayer (bin/trace_run) and bench.py all come through here.
 """
 from __future__ import annotations
 
@@ -22,7 +22,7 @@ def read_config(path: str) -> dict:
 # designs described layer by layer, served by RaggedEngine: architecture -> module with spec_from_config,
 # model_tensors and random_state_dict
 LAYERWISE = {"Sokevik": "sokevik", "Togalorn": "togalorn", "Fubepel": "fubepel", "Gimudra": "gimudra",
-             "Salizen": "salizen"}
+             "Salizen": "salizen", "Finezen": "finezen"}
 
 
 def family(cfg: dict) -> str:

@@ -598,17 +598,20 @@ def silu_mul(gu, out, bias=None, gelu=False):
 
 
 def attn_prep_append(proj, qbuf, k_cache, v_cache, row_ent, ent, page_table, H, G, D, V, rd, q_off, k_off, v_off,
-                     q_norm, k_norm, eps, cos_qk, sin_qk, cos_v, sin_v, bias=None, q_only=False, halves=False):
+                     q_norm, k_norm, eps, cos_qk, sin_qk, cos_v, sin_v, bias=None, q_only=False, halves=False, whole_norm=False):
     """q/k head norms, rotation and value rotation of a ragged step; q -> qbuf (float32), k / v -> the paged caches.
     bias float32 (indexed like proj's columns) is added first; q_only: no keys or values are made or appended (the caches
-    are only asked for their page size).  halves: rotation pairs (i, i + rd/2) instead of (2i, 2i+1)."""
+    are only asked for their page size).  halves: rotation pairs (i, i + rd/2) instead of (2i, 2i+1).  whole_norm: one norm
+    over all heads of q (k), with weights q_norm [H*D] (k_norm [G*D])."""
     _req(proj, proj.dtype), _req(k_cache, proj.dtype), _req(v_cache, proj.dtype)
     _f32(qbuf, q_norm, k_norm, cos_qk, sin_qk, cos_v, sin_v, bias), _i32(row_ent, ent, page_table)
+    if whole_norm and ((q_norm is not None and q_norm.numel() != H * D) or (k_norm is not None and k_norm.numel() != G * D)):
+        raise ValueError("attn_prep_append: a norm over the whole projection has a weight per row of it")
     tl = cos_qk.shape[0] if cos_qk is not None else (cos_v.shape[0] if cos_v is not None else 0)
     _call("dli_attn_prep_append", 1, _p(proj), _p(qbuf), _p(k_cache), _p(v_cache), _p(row_ent), _p(ent), _p(page_table),
           page_table.shape[1], k_cache.shape[2], proj.shape[0], H, G, D, V, rd, proj.shape[1], q_off, k_off, v_off,
           _p(q_norm), _p(k_norm), float(eps), _p(cos_qk), _p(sin_qk), _p(cos_v), _p(sin_v), tl, _dt(proj), _p(bias),
-          1 if q_only else 0, int(bool(halves)), _stream())
+          1 if q_only else 0, int(bool(halves)), int(bool(whole_norm)), _stream())
 
 
 def attn_ragged(qbuf, k_cache, v_cache, proj, out, row_ent, ent, page_table, H, G, D, V, scale, chunk=0, window=0,
@@ -716,11 +719,12 @@ def latent_q_absorb(q, uk, qbuf, row_ent, ent, cos_t, sin_t, H, D, R, K, halves=
     return qbuf
 
 
-def latent_v_up(o, uv, proj, out, H, V, K, g_off=-1):
-    """o [rows, H*K], uv [H*V, K] -> out [rows, H*V] = (uv[h] o[h]) * sigmoid(proj[:, g_off + h*V + v])."""
+def latent_v_up(o, uv, proj, out, H, V, K, g_off=-1, g_head=False):
+    """o [rows, H*K], uv [H*V, K] -> out [rows, H*V] = (uv[h] o[h]) * sigmoid(proj[:, g_off + h*V + v]); g_head: one gate
+    column per head, proj[:, g_off + h]."""
     _req(o, o.dtype), _req(uv, o.dtype), _req(out, o.dtype), _req(proj, o.dtype)
     _call("dli_latent_v_up", 1, _p(o), _p(uv), _p(proj), _p(out), o.shape[0], H, V, K,
-          proj.shape[1] if proj is not None else 0, g_off, _dt(o), _stream())
+          proj.shape[1] if proj is not None else 0, g_off, int(bool(g_head)), _dt(o), _stream())
     return out
 
 
@@ -779,28 +783,33 @@ def gated_group_rmsnorm(y, proj, w, out, groups, eps, z_off):
     return out
 
 
+_SCORES = {"softmax": 0, "sigmoid": 1}
+
+
 def moe_route(h, w_router, correction, wts, idw, sel_idx, sel_w, n_real, top, groups=1, keep=1, wscale=1.0, renorm=True,
-              logit_bias=None):
+              logit_bias=None, score="softmax", sg_w=None, sg=None):
     """Router of a mixture of experts on float32 rows: dense weights wts [rows, n_real], pass-through weight idw [rows],
     the choice sel_idx / sel_w [rows, top].  groups > 1: only outputs of the `keep` best of that many equal groups can be
     chosen; renorm False: the weights are the scores themselves; both times wscale.  logit_bias float32 [n_out]: added to
-    the logits (with renorm the weights are then the softmax over the chosen logits)."""
-    _f32(h, w_router, correction, wts, idw, sel_w, logit_bias), _i32(sel_idx)
+    the logits (with renorm the weights are then the softmax over the chosen logits).  score "sigmoid": scores are the
+    sigmoids of the logits.  sg_w float32 [d]: sg [rows] = sigmoid(h . sg_w), the shared expert's weight."""
+    _f32(h, w_router, correction, wts, idw, sel_w, logit_bias, sg_w, sg), _i32(sel_idx)
     _call("dli_moe_route", 1, _p(h), _p(w_router), _p(correction), _p(wts), _p(idw), _p(sel_idx), _p(sel_w), h.shape[0],
           h.shape[1], w_router.shape[0], int(n_real), int(top), int(groups), int(keep), float(wscale), 1 if renorm else 0,
-          _p(logit_bias), _stream())
+          _p(logit_bias), _SCORES[score], _p(sg_w), _p(sg), _stream())
 
 
 def _moe_mode(gated, silu):
     return 1 if not gated else (2 if silu else 0)
 
 
-def moe_act(gu, wts, act, n_exp, ff, limit, ff_s=0, limit_s=0.0, alpha=1.702, gated=True, silu=False):
+def moe_act(gu, wts, act, n_exp, ff, limit, ff_s=0, limit_s=0.0, alpha=1.702, gated=True, silu=False, weight_in=False, sg=None):
     """Activation of all experts' stacked projections, times the routing weights: the clamped gated form on [gate; up] rows,
-    (silu) silu(g) * u on them, or (gated False) max(u, 0)^2 on up rows alone."""
-    _req(gu, gu.dtype), _req(act, gu.dtype), _f32(wts)
+    (silu) silu(g) * u on them, or (gated False) max(u, 0)^2 on up rows alone.  weight_in: the weight is a factor on g and u
+    (the expert's input) instead; sg float32 [rows]: weight of the shared expert's output (None: 1)."""
+    _req(gu, gu.dtype), _req(act, gu.dtype), _f32(wts, sg)
     _call("dli_moe_act", 1, _p(gu), _p(wts), _p(act), gu.shape[0], int(n_exp), int(ff), float(limit), int(ff_s),
-          float(limit_s), float(alpha), gu.shape[1], _dt(gu), _moe_mode(gated, silu), _stream())
+          float(limit_s), float(alpha), gu.shape[1], _dt(gu), _moe_mode(gated, silu), int(bool(weight_in)), _p(sg), _stream())
     return act
 
 
@@ -808,17 +817,23 @@ def moe_sel_supported(d, ff, ff_s, top) -> bool:
     return bool(_lib.load().dli_moe_sel_supported(int(d), int(ff), int(ff_s), int(top)))
 
 
-def moe_sel(x, w_gu, w_down, sel_idx, sel_w, act_sel, y, n_exp, top, ff, limit, ff_s=0, limit_s=0.0, alpha=1.702, gated=True, silu=False):
+def moe_sel(x, w_gu, w_down, sel_idx, sel_w, act_sel, y, n_exp, top, ff, limit, ff_s=0, limit_s=0.0, alpha=1.702, gated=True, silu=False,
+            weight_in=False, sg=None):
     """Few rows (decode): the chosen experts' and the shared expert's weights only -> y [rows, d] (bf16)."""
-    _req(x), _req(w_gu), _req(w_down), _req(act_sel), _req(y), _i32(sel_idx), _f32(sel_w)
+    _req(x), _req(w_gu), _req(w_down), _req(act_sel), _req(y), _i32(sel_idx), _f32(sel_w, sg)
     _call("dli_moe_sel_bf16", 2, _p(x), _p(w_gu), _p(w_down), _p(sel_idx), _p(sel_w), _p(act_sel), _p(y), x.shape[0],
           x.shape[1], int(n_exp), int(top), int(ff), float(limit), int(ff_s), float(limit_s), float(alpha),
-          _moe_mode(gated, silu), _stream())
+          _moe_mode(gated, silu), int(bool(weight_in)), _p(sg), _stream())
     return y
 
 
 # ---------------------------------------------------------------------------------------------------------------
 # Pre-norm layers with layer scale, token shift and depth average (prenorm_rows.cu)
+def _plain_scores(r, name):
+    if r.get("score", "softmax") != "softmax" or r.get("sg_w") is not None:
+        raise ValueError(f"{name}: its router has softmax scores and no gate of a shared expert")
+
+
 def layer_close(x, y=None, bias=None, idw=None, h_in=None, ls=None, xs=None, n_prev=0, dwa=None, w_next=None, shift=None,
                 tail=None, ent=None, out_f=None, out_e=None, eps: float = 1e-6, route=None):
     """x += ls * (y + bias + idw[:, None] * h_in) (x float32 in place; y in the element type); with dwa (float32 [n_prev + 1])
@@ -831,6 +846,7 @@ def layer_close(x, y=None, bias=None, idw=None, h_in=None, ls=None, xs=None, n_p
     r = route or {}
     if route is not None:
         _f32(r["w_router"], r.get("correction"), r.get("logit_bias"), r["wts"], r["idw"], r["sel_w"]), _i32(r["sel_idx"])
+        _plain_scores(r, "layer_close")
         if out_f is None or r["w_router"].shape[1] != x.shape[1]:
             raise ValueError("layer_close: the router reads the float32 normed rows")
     for t in (y, out_e):
@@ -929,6 +945,7 @@ def streams_close(x, rows, y=None, mix=None, outw=None, in_next=None, w_next=Non
     r = route or {}
     if route is not None:
         _f32(r["w_router"], r.get("correction"), r.get("logit_bias"), r["wts"], r["idw"], r["sel_w"]), _i32(r["sel_idx"])
+        _plain_scores(r, "streams_close")
         if r["w_router"].shape[1] != x.shape[2]:
             raise ValueError("streams_close: the router reads the normed rows")
     for t in (y, out_e):
@@ -943,6 +960,37 @@ def streams_close(x, rows, y=None, mix=None, outw=None, in_next=None, w_next=Non
           _p(r.get("sel_w")), r["w_router"].shape[0] if route is not None else 0, int(r.get("n_real", 0)), int(r.get("top", 0)),
           int(r.get("groups", 1)), int(r.get("keep", 1)), float(r.get("wscale", 1.0)), 1 if r.get("renorm", True) else 0,
           _stream())
+    return x
+
+
+# ---------------------------------------------------------------------------------------------------------------
+# Layers whose norms are dynamic tanh maps (dyn_tanh_rows.cu); a map is (w float32 [d], b float32 [d], alpha)
+def dyn_tanh_close(x, y=None, post=None, mult: float = 1.0, add=None, nxt=None, out_f=None, out_e=None, route=None):
+    """x float32 [rows, d] in place: with y (element type) x += mult * (tanh(alpha y) * w + b) of the map `post`, then x += add
+    (float32); the map `nxt` of the new x -> out_f (float32) / out_e (element type).  route: moe_route's arguments after h as a
+    dict; the router runs on those rows in the same kernel."""
+    pw, pb, pa = post if post is not None else (None, None, 0.0)
+    nw, nb, na = nxt if nxt is not None else (None, None, 0.0)
+    r = route or {}
+    _f32(x, pw, pb, add, nw, nb, out_f)
+    if route is not None:
+        _f32(r["w_router"], r.get("correction"), r.get("logit_bias"), r["wts"], r["idw"], r["sel_w"], r.get("sg_w"), r.get("sg"))
+        _i32(r["sel_idx"])
+        if r["w_router"].shape[1] != x.shape[1]:
+            raise ValueError("dyn_tanh_close: the router reads the mapped rows")
+    for t in (y, out_e):
+        if t is not None:
+            _req(t, t.dtype)
+    for t in (pw, pb, nw, nb):
+        if t is not None and t.numel() != x.shape[1]:
+            raise ValueError("dyn_tanh_close: a map has a weight and an offset per channel")
+    ref = y if y is not None else out_e
+    _call("dli_dyn_tanh_close", 1, _p(y), _p(pw), _p(pb), float(pa), float(mult), _p(add), _p(x), _p(nw), _p(nb), float(na), _p(out_f),
+          _p(out_e), x.shape[0], x.shape[1], _dt(ref) if ref is not None else 1, _p(r.get("w_router")), _p(r.get("logit_bias")),
+          _p(r.get("correction")), _p(r.get("wts")), _p(r.get("idw")), _p(r.get("sel_idx")), _p(r.get("sel_w")),
+          r["w_router"].shape[0] if route is not None else 0, int(r.get("n_real", 0)), int(r.get("top", 0)), int(r.get("groups", 1)),
+          int(r.get("keep", 1)), float(r.get("wscale", 1.0)), 1 if r.get("renorm", True) else 0, _SCORES[r.get("score", "softmax")],
+          _p(r.get("sg_w")), _p(r.get("sg")), _stream())
     return x
 
 

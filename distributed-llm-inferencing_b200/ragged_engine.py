@@ -4,13 +4,13 @@ ShardEngine (engine.py) serves uniform Llama / GPT-2 stacks on rectangular batch
 This engine serves stacks described layer by layer (HybridSpec): every layer has a token mixer — softmax attention
 with its options, latent attention, a recurrent cell with a matrix state (mLSTM, state-space, gated delta rule, linear
 attention with a fixed or an input-made decay), or two of these side by side on one input — and optionally a
-feed-forward (dense or a mixture of experts).  Five layer styles: sublayers in sequence, each
+feed-forward (dense or a mixture of experts).  Six layer styles: sublayers in sequence, each
 wrapped in a pre-norm and a post-norm with one weight and reading its input through a short causal convolution;
 mixer and feed-forward side by side on one grouped norm; sublayers that read the residual stream itself and are
 normed on their output only, followed by a per-layer token input; pre-normed sublayers with a weight vector per
 norm, a layer scale on each result, a token shift in front of the mixer and an average over all layers' results
 after the layer; pre-normed sublayers that read a weighted sum of several residual streams and mix all of them
-afterwards.  Layers may share another layer's weights while
+afterwards; sublayers between two dynamic tanh maps instead of norms.  Layers may share another layer's weights while
 keeping a cache / state of their own, or read another layer's cache.  The residual stream, norms, rotation
 angles, scores, softmax weights, convolution and recurrent state are fp32; projections run in the element type of the
 engine (bf16 on the tcgen05 / GEMV kernels of ops.linear, or float32 on the CUDA-core GEMM).
@@ -50,11 +50,13 @@ class MixerSpec:
     scale: float = 1.0
     rot_dims: int = 0              # leading dims of q / k that are rotated (interleaved pairs); 0 = none
     rot_base: float = 10000.0
-    rot_scaling: Optional[dict] = None   # {factor, low, high, original}: wavelength-dependent frequency scaling
+    rot_scaling: Optional[dict] = None   # {factor, low, high, original}: wavelength-dependent frequency scaling, or
+                                   # {factor, original, fast, slow}: scaling by pair number with a gain (YaRN)
     chunk: int = 0                 # > 0: a position sees only its own block of `chunk` positions
     window: int = 0                # > 0: a position sees the last `window` positions
     keep_first: int = 0            # with a chunk or window: the first `keep_first` positions stay visible
     qk_norm: bool = False          # per-head RMS norm of q and k (weights q_norm / k_norm; without them: plain division)
+    qk_norm_whole: bool = False    # the norm runs over the whole query (key) projection, a weight per row of it
     rotate_values: bool = False    # values rotated by their position, outputs turned back by theirs
     sink: bool = False             # one extra softmax term per head without key or value
     head_gate: bool = False        # sigmoid gate per head on the output
@@ -128,6 +130,9 @@ class MoESpec:
     renorm: bool = True            # weights divided by the sum of the chosen scores (False: the scores themselves)
     act: str = "clamp"             # gated experts: the clamped form above, or "silu" (silu(g) * u)
     router_bias: bool = False      # the router's logits have a bias
+    score: str = "softmax"         # scores of the router's logits, or "sigmoid" (each logit alone)
+    weight_in: bool = False        # the routing weight scales the expert's input instead of its output
+    shared_gate: bool = False      # the shared expert's output times sigmoid(one more router row . input)
 
     @property
     def total_ff(self) -> int:
@@ -144,6 +149,7 @@ class LayerSpec:
                                    # read it and x += mixer + feed-forward.  False: pre-/post-normed sublayers in sequence
     ckpt: Optional[int] = None     # the checkpoint's layer number when it differs from the position in `layers`
     reenter: Optional[int] = None  # t: before this layer x <- W_loop [x | embedding output] + step[t]
+    add_embedding: bool = False    # before this layer the embedding output is added to x
     post_only: bool = False        # True: sublayers read x itself and x += rmsnorm(sublayer(x)) * weight vector; no input
                                    # convolution
     ff_limit: float = 0.0          # > 0: the dense feed-forward is min(g, limit) sigmoid(alpha min(g, limit)) (clamp(u) + 1)
@@ -174,6 +180,9 @@ class HybridSpec:
     pos_base: float = 10000.0
     streams: int = 0               # > 0: that many residual streams (every layer pre_norm): a sublayer reads
                                    # u = sum_s in[s] x_s, then x_t <- sum_s mix[s, t] x_s + out[t] * result
+    norm_fn: str = "rms"           # "tanh": every norm is a map tanh(alpha z) * w + b per channel, sublayers (every layer pre_norm)
+                                   # have one before and one after them: x += residual_mult * map'(sublayer(map(x)))
+    residual_mult: float = 1.0
     bigram: Optional[tuple] = None  # (buckets, mul_prev, mul_cur): a table row of the hashed pair (previous token, token) is
                                    # added to the embedding
 
@@ -187,12 +196,23 @@ class HybridSpec:
 
 
 def rot_frequencies(base: float, dims: int, scaling: Optional[dict]) -> torch.Tensor:
-    """float64 [dims/2]: f_i = base^(-2i/dims), then the wavelength-dependent scaling of long-context Llama
-    checkpoints: wavelengths below original/high keep f, above original/low use f/factor, between them a linear
-    blend in original/wavelength."""
+    """float64 [dims/2]: f_i = base^(-2i/dims), then, with {factor, low, high, original}, the wavelength-dependent scaling of
+    long-context Llama checkpoints: wavelengths below original/high keep f, above original/low use f/factor, between them a
+    linear blend in original/wavelength.  With {factor, original, fast, slow} the blend is linear in the pair number, from
+    the pair that turns `fast` times over `original` positions (f) to the one that turns `slow` times (f/factor), those two
+    rounded outwards to whole pairs."""
     f = torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)
     if not scaling:
         return f
+    if "fast" in scaling:
+        fac, orig = float(scaling["factor"]), float(scaling["original"])
+
+        def pair(turns):
+            return dims * math.log(orig / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+        lo, hi = max(math.floor(pair(float(scaling["fast"]))), 0), min(math.ceil(pair(float(scaling["slow"]))), dims - 1)
+        ramp = ((torch.arange(dims // 2, dtype=torch.float64) - lo) / max(hi - lo, 1e-3)).clamp(0.0, 1.0)
+        return f / fac * ramp + f * (1.0 - ramp)
     fac, lo, hi, orig = (float(scaling[k]) for k in ("factor", "low", "high", "original"))
     out = []
     for fi in f.tolist():
@@ -205,6 +225,11 @@ def rot_frequencies(base: float, dims: int, scaling: Optional[dict]) -> torch.Te
             s = (orig / wl - lo) / (hi - lo)
             out.append((1.0 - s) * fi / fac + s * fi)
     return torch.tensor(out, dtype=torch.float64)
+
+
+def rot_gain(scaling: Optional[dict]) -> float:
+    """Factor on cosine and sine: 1 + 0.1 ln(factor) with the pair-number scaling, else 1."""
+    return 0.1 * math.log(float(scaling["factor"])) + 1.0 if scaling and "fast" in scaling else 1.0
 
 
 def _ceil(a: int, b: int) -> int:
@@ -238,6 +263,9 @@ class RaggedEngine:
         self.slots = StateSlots(self.max_batch, self.device)
         if spec.streams and not all(L.pre_norm and not (L.token_shift or L.layer_scale or L.depth_avg) for L in spec.layers):
             raise ValueError("several residual streams: every layer pre-normed, without shift, layer scale or average")
+        if spec.norm_fn not in ("rms", "tanh") or (spec.norm_fn == "tanh" and (spec.streams or not all(
+                L.pre_norm and not (L.token_shift or L.layer_scale or L.depth_avg or L.ff_bias) for L in spec.layers))):
+            raise ValueError("norms as tanh maps: one stream, every layer pre-normed, without shift, layer scale, average or biases")
         if spec.bigram:
             self.slots.add(("last",), dtype=torch.int32)       # the sequence's last token
         for i, L in enumerate(spec.layers):
@@ -296,13 +324,15 @@ class RaggedEngine:
 
     # ------------------------------------------------------------------ weights
     def _table(self, base: float, dims: int, scaling: Optional[dict]):
-        """fp32 cos / sin [max_seq_len, dims/2] of position * frequency, angles taken in float64 on the host."""
+        """fp32 cos / sin [max_seq_len, dims/2] of position * frequency (times the scaling's gain), angles taken in float64 on
+        the host."""
         key = (base, dims, tuple(sorted(scaling.items())) if scaling else None)
         if key not in self._tables:
             f = rot_frequencies(base, dims, scaling)
             ang = torch.arange(self.max_seq_len, dtype=torch.float64)[:, None] * f[None, :]
-            self._tables[key] = (ang.cos().float().contiguous().to(self.device),
-                                 ang.sin().float().contiguous().to(self.device))
+            gain = rot_gain(scaling)
+            self._tables[key] = ((gain * ang.cos()).float().contiguous().to(self.device),
+                                 (gain * ang.sin()).float().contiguous().to(self.device))
         return self._tables[key]
 
     def load_tensors(self, t: dict) -> None:
@@ -327,6 +357,8 @@ class RaggedEngine:
 
         self.w = {"embed": t["embed"].to(E).contiguous().to(dev), "head": mat(t["head"]),
                   "final_norm": vec(t["final_norm"]) if s.norm_groups else float(t["final_norm"])}
+        if s.norm_fn == "tanh":
+            self.w["final_norm"] = (vec(t["final_norm"]), vec(t["final_norm_b"]), float(t["final_norm_a"]))
         if s.bigram:
             self.w["bigram"] = t["bigram"].to(E).contiguous().to(dev)
         if s.side_width:
@@ -345,6 +377,8 @@ class RaggedEngine:
             g = at + qn + kn + (0 if m.keys_as_values else vn)
             # a norm without weights is the norm with unit weights; values that are the keys share their columns
             ones = torch.ones(m.dim, dtype=torch.float32, device=dev)
+            if m.qk_norm_whole and not ("q_norm" in src and "k_norm" in src):
+                raise ValueError("a norm over the whole query / key projection needs its weights")
             sink = vec(src["sink"]) if m.sink else (torch.zeros(m.heads, dtype=torch.float32, device=dev) if m.zero_sink else None)
             return ws, {"off": {"q": at, "k": at + qn, "v": at + qn + (0 if m.keys_as_values else kn),
                                 "g": g if m.head_gate or m.out_gate else -1},
@@ -417,10 +451,10 @@ class RaggedEngine:
                     raise ValueError(f"layer {i}: a query latent together with another layer's cache is not supported")
                 nq = m.q_rank if m.q_rank else m.heads * (m.dim + m.rot_dims)
                 parts = [src["dq"] if m.q_rank else src["q"]] + ([src["dkv"]] if m.kv_from is None else []) + \
-                        ([src["g"]] if m.out_gate else [])
+                        ([src["g"]] if m.out_gate or m.head_gate else [])
                 d["w_proj"] = mat(*parts)
                 nkv = m.kv_rank + m.rot_dims if m.kv_from is None else 0
-                d["off"] = {"cq": 0, "kv": nq, "g": nq + nkv if m.out_gate else -1}
+                d["off"] = {"cq": 0, "kv": nq, "g": nq + nkv if m.out_gate or m.head_gate else -1}
                 if m.q_rank:
                     d["w_uq"] = mat(src["uq"], pad_rows=False)
                     d["q_norm"] = vec(src["dq_norm"])
@@ -468,6 +502,9 @@ class RaggedEngine:
                     raise ValueError(f"layer {i}: {d['dwa'].numel()} averaging weights for {i + 2} results")
                 if L.ff or L.moe is not None:
                     d["norm2"] = vec(src["norm2"])
+                if s.norm_fn == "tanh":
+                    for k in ("norm1", "norm1b", "norm2", "norm2b") if (L.ff or L.moe is not None) else ("norm1", "norm1b"):
+                        d[k] = (vec(src[k]), vec(src[k + "_b"]), float(src[k + "_a"]))
             if L.ff and L.pre_norm:
                 # silu(gate) * up as the GEMM's epilogue where there are no biases and the tile's alignment holds; else
                 # [gate rows | up rows] and the activation (with the biases) as a kernel of its own
@@ -515,6 +552,7 @@ class RaggedEngine:
                 d["w_down"] = torch.cat([x.to(E) for x in downs], dim=1).contiguous().to(dev)
                 d["w_router"], d["corr"] = f32(src["router"]), vec(src["correction"]) if "correction" in src else None
                 d["router_b"] = vec(src["router_b"]) if e.router_bias else None
+                d["shared_g"] = vec(src["shared_g"]) if e.shared_gate else None
             self.layers[i] = d
 
     def weight_bytes(self) -> int:
@@ -612,10 +650,12 @@ class RaggedEngine:
         if moes:
             self._wts = torch.empty(rows * max(e.experts for e in moes), dtype=f32, device=dev)
             self._idw = torch.empty(rows, dtype=f32, device=dev)
+            self._shw = torch.empty(rows, dtype=f32, device=dev)
             self._sel_idx = torch.empty(rows * max(e.top for e in moes), dtype=torch.int32, device=dev)
             self._sel_w = torch.empty(rows * max(e.top for e in moes), dtype=f32, device=dev)
-        if s.loop_passes:
+        if s.loop_passes or any(L.add_embedding for L in s.layers):
             self._x0 = torch.empty(rows, s.width, dtype=f32, device=dev)
+        if s.loop_passes:
             self._cat = torch.empty(rows, 2 * s.width, dtype=E, device=dev)
         self._hw = torch.empty(max(self.max_batch, 8), s.width, dtype=E, device=dev)
         self._ws_rows = rows
@@ -681,6 +721,7 @@ class RaggedEngine:
             used = [p for slot, toks in batch
                     for p in self.kv.owned[slot][:(self.lengths[slot] + len(toks) + self.kv.page_size - 1) // self.kv.page_size]]
             self._step_pages = (min(used), max(used))
+            self._step_spans = [(slot, self.lengths[slot], self.lengths[slot] + len(toks)) for slot, toks in batch]
         # steps that hold a portion of a prompt run attention in 64-row query tiles on the tensor cores
         tiles: List[int] = []
         if any(len(t) >= self.tc_min_rows for _, t in batch):
@@ -763,6 +804,9 @@ class RaggedEngine:
         y = self._y[:rows]
         if s.streams:
             self._stream_layers(rows, nw, views, long_step, tiles)
+            return self._head(self._hs[:rows], d_want, nw, logits_out)
+        if s.norm_fn == "tanh":
+            self._tanh_layers(rows, nw, views, tiles)
             return self._head(self._hs[:rows], d_want, nw, logits_out)
         single = rows == n_ent and s.taps > 1 and self.layer_trace is None  # decode rows: norm + convolution fused
 
@@ -1051,6 +1095,7 @@ class RaggedEngine:
     def _route_args(self, e, P, rows):
         """Arguments of the router for kernels that run it on a row they have just normed."""
         return dict(w_router=P["w_router"], correction=P["corr"], logit_bias=P["router_b"],
+                    score=e.score, sg_w=P["shared_g"], sg=self._shw[:rows] if e.shared_gate else None,
                     wts=self._wts[:rows * e.experts].view(rows, e.experts), idw=self._idw[:rows],
                     sel_idx=self._sel_idx[:rows * e.top].view(rows, e.top), sel_w=self._sel_w[:rows * e.top].view(rows, e.top),
                     n_real=e.experts, top=e.top, groups=e.groups, keep=e.keep, wscale=e.route_scale, renorm=e.renorm)
@@ -1058,18 +1103,18 @@ class RaggedEngine:
     def _experts(self, e, P, he, route, y):
         """y = the weighted sum of the chosen experts' (and the shared expert's) outputs for the rows he."""
         rows = he.shape[0]
-        silu = e.act == "silu"
+        more = dict(gated=e.gated, silu=e.act == "silu", weight_in=e.weight_in, sg=route["sg"])
         if self._moe_sel_ok(e, rows):
             # decode rows of a sparse enough mixture: stream only the chosen experts' weights
             n_sel = e.top * e.ff + e.shared_ff
             ops.moe_sel(he, P["w_gu"], P["w_down"], route["sel_idx"], route["sel_w"], self._act[:rows * n_sel].view(rows, n_sel), y,
-                        e.experts, e.top, e.ff, e.limit, e.shared_ff, e.shared_limit, e.alpha, gated=e.gated, silu=silu)
+                        e.experts, e.top, e.ff, e.limit, e.shared_ff, e.shared_limit, e.alpha, **more)
             return
         n_gu = P["w_gu"].shape[0]
         gu = self._gu[:rows * n_gu].view(rows, n_gu)
         self._lin(he, P["w_gu"], gu)
         act = self._act[:rows * e.total_ff].view(rows, e.total_ff)
-        ops.moe_act(gu, route["wts"], act, e.experts, e.ff, e.limit, e.shared_ff, e.shared_limit, e.alpha, gated=e.gated, silu=silu)
+        ops.moe_act(gu, route["wts"], act, e.experts, e.ff, e.limit, e.shared_ff, e.shared_limit, e.alpha, **more)
         self._lin(act, P["w_down"], y)
 
     # ------------------------------------------------------------------ layers with several residual streams
@@ -1122,6 +1167,54 @@ class RaggedEngine:
             if self.layer_trace is not None:
                 self.layer_trace.append(xst[:, :rows].sum(0))
 
+    # ------------------------------------------------------------------ layers with tanh maps instead of norms
+    def _tanh_layers(self, rows, nw, views, tiles):
+        """All layers of a model whose norms are tanh maps, from the embedding to the last map (rows in _hs).  Between two
+        projections ONE elementwise kernel (ops.dyn_tanh_close): the map of the sublayer's result, the scaled residual add, the
+        embedding output in front of a loop's next pass, the next sublayer's map and, before a mixture of experts, the router."""
+        s = self.spec
+        d_tok, d_rent, d_ent, d_want, d_tiles = views
+        x, he, y = self._x[:rows], self._he[:rows], self._y[:rows]
+        x0 = self._x0[:rows] if any(L.add_embedding for L in s.layers) else None
+        ops.embedding_f32(d_tok, self.w["embed"], x, s.embed_scale, out2=x0)
+        ops.dyn_tanh_close(x, nxt=self.layers[s.source(0)]["norm1"], out_e=he)
+        for li, L in enumerate(s.layers):
+            P, m = self.layers[s.source(li)], L.mixer
+            n_proj, n_mix = P["w_proj"].shape[0], m.out_width
+            proj = self._proj[:rows * n_proj].view(rows, n_proj)
+            mix = self._mix[:rows * n_mix].view(rows, n_mix)
+            self._lin(he, P["w_proj"], proj)
+            if m.kind == "attention":
+                self._attention(li, m, P, proj, mix, rows, views, tiles)
+            elif m.kind == "latent_attention":
+                self._latent_attention(li, m, P, proj, mix, rows, views, tiles)
+            else:
+                raise ValueError(f"layer {li}: mixer {m.kind!r} has no form between tanh maps")
+            self._lin(mix, P["wo"], y)
+            post = P["norm1b"]
+            if L.ff or L.moe is not None:
+                route = self._route_args(L.moe, P, rows) if L.moe is not None else None
+                ops.dyn_tanh_close(x, y, post, s.residual_mult, nxt=P["norm2"], out_e=he, route=route)
+                if L.moe is not None:
+                    self._experts(L.moe, P, he, route, y)
+                else:
+                    self._dense_ff(L, P, he, y)
+                post = P["norm2b"]
+            if li + 1 == s.n_layers:
+                add, nxt = None, dict(nxt=self.w["final_norm"], out_f=self._hs[:rows]) if nw else {}
+            else:
+                add = x0 if s.layers[li + 1].add_embedding else None
+                nxt = dict(nxt=self.layers[s.source(li + 1)]["norm1"], out_e=he)
+            if self.layer_trace is not None and add is not None:
+                # debugging: the residual stream as the layer leaves it, before the next pass adds to it
+                ops.dyn_tanh_close(x, y, post, s.residual_mult)
+                self.layer_trace.append(x.clone())
+                ops.dyn_tanh_close(x, add=add, **nxt)
+                continue
+            ops.dyn_tanh_close(x, y, post, s.residual_mult, add=add, **nxt)
+            if self.layer_trace is not None:
+                self.layer_trace.append(x.clone())
+
     def _linear_attention(self, li, m, P, proj, mix, rows, views, long_step):
         """Linear attention with a decaying state: the recurrence over the state slot (row by row, or as small matrix
         products for steps with portions of prompts), then the norm of the outputs and the gate."""
@@ -1162,7 +1255,8 @@ class RaggedEngine:
         more = dict(cap=m.softcap, g_chan=m.out_gate, out_scale=m.out_scale)
         ops.attn_prep_append(proj, qbuf, kc, vc, d_rent, d_ent, pt, m.heads, m.kv_heads, m.dim, m.vdim,
                              m.rot_dims, off["q"], off["k"], off["v"], P["q_norm"], P["k_norm"], s.eps,
-                             cq, sq, cv, sv, bias=P.get("qkv_b"), q_only=m.kv_from is not None, halves=m.rot_halves)
+                             cq, sq, cv, sv, bias=P.get("qkv_b"), q_only=m.kv_from is not None, halves=m.rot_halves,
+                             whole_norm=m.qk_norm_whole)
         if tiles and m.scale > 0 and ops.attn_ragged_tc_supported(m.dim, m.vdim, E):
             ops.attn_ragged_tc(qbuf, kc, vc, proj, mix, d_ent, d_tiles, pt, m.heads, m.kv_heads, m.dim, m.vdim,
                                m.scale, chunk=m.chunk, window=m.window, sink=P["sink"], g_off=off["g"],
@@ -1263,8 +1357,9 @@ class RaggedEngine:
             q = proj[:, :H * (D + R)]  # the queries are the leading columns of the projection
         sink = P.get("sink")
         ps = self.kv.page_size
+        gated = m.out_gate or m.head_gate
         if tiles and "w_ukv" in P and m.scale > 0 and self._step_pages is not None and (K + R) % 8 == 0:
-            lo, hi = self._step_pages
+            lo, hi = self._pages_in_view(m.window)
             n = (hi - lo + 1) * ps
             need = n * H * (2 * D + R + 2 * V)
             if need <= self.latent_expand_max_elems:
@@ -1278,8 +1373,8 @@ class RaggedEngine:
                 ops.latent_expand(kvx, rows_pool, kx, vx, H, D, R, V, K, ps)
                 qbuf = self._qbuf[:rows * H * (D + R)].view(rows, H * (D + R))
                 ops.latent_q_absorb(q, None, qbuf, d_rent, d_ent, cos_t, sin_t, H, D, R, D, halves=hv)
-                ops.attn_ragged_tc(qbuf, kx, vx, None, mix, d_ent, d_tiles, self.kv.page_table, H, H, D + R, V, m.scale,
-                                   page_base=lo, sink=sink)
+                ops.attn_ragged_tc(qbuf, kx, vx, proj if m.head_gate else None, mix, d_ent, d_tiles, self.kv.page_table, H, H, D + R, V,
+                                   m.scale, page_base=lo, sink=sink, window=m.window, g_off=off["g"] if m.head_gate else -1)
                 if m.out_gate:
                     ops.sigmoid_gate(mix, proj, off["g"])
                 return
@@ -1290,10 +1385,22 @@ class RaggedEngine:
         # count depends on the rows alone (a replayed graph keeps it while the contexts grow)
         # (heads in fours: the shared-key/value kernel gives a CTA four heads of a row)
         splits = max(1, min(64, (4 * self._sms) // (rows * ((H + 3) // 4)))) if rows <= 16 else 1
+        if m.window:
+            splits = max(1, min(splits, (m.window + 31) // 32))
         part = self._apart if splits > 1 else None
         ops.attn_ragged(qbuf, pool, pool, None, olat, d_rent, d_ent, self.kv.page_table, H, 1, K + R, K, m.scale,
-                        ldv=K + R, splits=splits, part=part, sink=sink)
-        ops.latent_v_up(olat, P["uv"], proj if m.out_gate else None, mix, H, V, K, g_off=off["g"])
+                        ldv=K + R, splits=splits, part=part, sink=sink, window=m.window)
+        ops.latent_v_up(olat, P["uv"], proj if gated else None, mix, H, V, K, g_off=off["g"], g_head=m.head_gate)
+
+    def _pages_in_view(self, window):
+        """First and last pool page that the step's rows read: whole sequences, or, with a window, from the 64-position tile
+        that holds the first row's oldest visible key."""
+        if not window:
+            return self._step_pages
+        ps = self.kv.page_size
+        used = [p for slot, start, end in self._step_spans
+                for p in self.kv.owned[slot][max(0, start - window + 1) // 64 * 64 // ps:(end + ps - 1) // ps]]
+        return min(used), max(used)
 
     def _mamba2(self, li, m, P, proj, mix, rows, views, long_step=False):
         d_tok, d_rent, d_ent, d_want, d_tiles = views

@@ -475,12 +475,13 @@ int dli_silu_mul(const void* gu, void* act, int M, int F, int ld, int dt, const 
  * both NULL): the distance penalty r1[h] * ln(1 + r2[h] * (i - j)) is taken off the scaled score of query i, key j.
  * halves: rotation pairs (i, i + rd/2) instead of (2i, 2i+1).  cap > 0: scaled scores become cap * tanh(score / cap).
  * g_chan: the gate has a column per output channel, proj[row, g_off + h*V + v].  out_scale: a factor on the output.  ldo:
- * elements between output rows (0 = H*V), for outputs that are a part of wider rows. */
+ * elements between output rows (0 = H*V), for outputs that are a part of wider rows.  whole_norm: ONE norm over all heads
+ * of the query (key) projection, q_norm [H*D] and k_norm [G*D]. */
 int dli_attn_prep_append(const void* proj, float* qbuf, void* k_cache, void* v_cache, const int32_t* row_ent,
                          const int32_t* ent, const int32_t* page_table, int max_pages, int page_size, int rows, int H,
                          int G, int D, int V, int rd, int ldp, int q_off, int k_off, int v_off, const float* q_norm,
                          const float* k_norm, float eps, const float* cos_qk, const float* sin_qk, const float* cos_v,
-                         const float* sin_v, int table_len, int dt, const float* bias, int q_only, int halves,
+                         const float* sin_v, int table_len, int dt, const float* bias, int q_only, int halves, int whole_norm,
                          dli_stream_t stream);
 int dli_attn_ragged(const float* qbuf, const void* k_cache, const void* v_cache, const void* proj, void* out,
                     const int32_t* row_ent, const int32_t* ent, const int32_t* page_table, int max_pages, int page_size,
@@ -490,7 +491,8 @@ int dli_attn_ragged(const float* qbuf, const void* k_cache, const void* v_cache,
 
 /* The same attention for steps that hold portions of prompts, on the tensor cores (bf16 caches only): one CTA per
  * 64-row query tile of an entry and query head; tiles[2t] = entry, tiles[2t+1] = first row of the tile within the
- * entry.  dli_attn_ragged_tc_supported says whether (key size, value size, element type) has a tile. */
+ * entry.  dli_attn_ragged_tc_supported says whether (key size, value size, element type) has a tile: bf16, multiples of 8
+ * from 32 up to 128 / 256 (sizes between the tiles' run in the next larger one). */
 int dli_attn_ragged_tc_supported(int D, int V, int dt);
 int dli_attn_ragged_tc(const float* qbuf, const void* k_cache, const void* v_cache, const void* proj, void* out,
                        const int32_t* ent, const int32_t* tiles, int n_tiles, const int32_t* page_table, int max_pages,
@@ -523,7 +525,8 @@ int dli_mlstm_ragged_parallel(const void* proj, float* o_scratch, void* y, const
  * -> cq [rows, Q]; c = rmsnorm(proj[kv_off : +K]) * kv_norm and k_r = rot(proj[kv_off + K : +R]) -> the pool.
  * dli_latent_q_absorb: q [rows, H, D + R] and uk [H*D, K] -> qbuf [rows, H, K + R] fp32 = [uk[h]^T q_n | rot(q_r)], so
  * that dli_attn_ragged over the pool (G = 1, key size K + R, value size K, ldv = K + R) gives each head's output in
- * the latent; dli_latent_v_up: out [rows, H*V] = (uv[h] o[row, h]) * sigmoid(proj[row, g_off + h*V + v]).
+ * the latent; dli_latent_v_up: out [rows, H*V] = (uv[h] o[row, h]) * sigmoid(proj[row, g_off + h*V + v]), with g_head one
+ * gate column per head, sigmoid(proj[row, g_off + h]).
  * Q == 0: the model has no query latent and that part is skipped (cq, q_norm may be NULL).  halves: pair i of a
  * rotated part is entries (2i, 2i+1) when 0, entries (i, i + R/2) otherwise.  ldq: elements between the rows of q
  * (0 = H * (D + R)). */
@@ -535,7 +538,7 @@ int dli_latent_q_absorb(const void* q, const void* uk, float* qbuf, const int32_
                         const float* cos_t, const float* sin_t, int rows, int H, int D, int R, int K, int halves, int ldq,
                         int dt, dli_stream_t stream);
 int dli_latent_v_up(const void* o, const void* uv, const void* proj, void* out, int rows, int H, int V, int K, int ldp,
-                    int g_off, int dt, dli_stream_t stream);
+                    int g_off, int g_head, int dt, dli_stream_t stream);
 /* Steps with portions of prompts run latent attention head by head on the tensor cores instead: kv [n, H*D + H*V] =
  * the up-projections of n consecutive pool rows (n a multiple of page_size), pool [n, K + R] those rows ->
  * kx [n / page_size, H, page_size, D + R] = [k_n | k_r] and vx [.., V], the layout of dli_attn_ragged_tc;
@@ -577,12 +580,14 @@ int dli_gated_group_rmsnorm(const float* y, const void* proj, const float* w, vo
  * themselves; both forms times wscale.  mode 1 (dli_moe_act, dli_moe_sel_bf16): experts without a gate,
  * act = max(u, 0)^2 * weight on gu [rows, ld] = the experts' stacked up projections [ff each], then the shared one's.
  * mode 2: silu(g) * u * weight, no limits.  logit_bias [n_out] or NULL is added to the logits; with renorm 1 the weights
- * are then the softmax over the chosen logits alone. */
+ * are then the softmax over the chosen logits alone.  score 1: the scores are a sigmoid of each logit instead.  sg_w [d] or
+ * NULL: sg[row] = sigmoid(h . sg_w), a weight of the shared expert's output (dli_moe_act / dli_moe_sel_bf16: sg or NULL = 1).
+ * w_in != 0: the routing weight scales the routed experts' INPUT (a factor on g and u) instead of their output. */
 int dli_moe_route(const float* h, const float* w_router, const float* correction, float* wts, float* idw, int32_t* sel_idx,
                   float* sel_w, int rows, int d, int n_out, int n_real, int top, int groups, int keep, float wscale,
-                  int renorm, const float* logit_bias, dli_stream_t stream);
+                  int renorm, const float* logit_bias, int score, const float* sg_w, float* sg, dli_stream_t stream);
 int dli_moe_act(const void* gu, const float* wts, void* act, int rows, int n_exp, int ff, float limit, int ff_s,
-                float limit_s, float alpha, int ld, int dt, int mode, dli_stream_t stream);
+                float limit_s, float alpha, int ld, int dt, int mode, int w_in, const float* sg, dli_stream_t stream);
 /* Few rows (decode steps, bf16): only the weights of each row's chosen experts (and the shared expert) are read.
  * x [rows, d]; w_gu and w_down in the stacked layout of dli_moe_act ([gate; up] per expert, shared last;
  * w_down [d, n_exp*ff + ff_s]); act_sel [rows, top*ff + ff_s] scratch; y [rows, d] = the weighted sum of the chosen
@@ -590,7 +595,7 @@ int dli_moe_act(const void* gu, const float* wts, void* act, int rows, int n_exp
 int dli_moe_sel_supported(int d, int ff, int ff_s, int top);
 int dli_moe_sel_bf16(const void* x, const void* w_gu, const void* w_down, const int32_t* sel_idx, const float* sel_w,
                      void* act_sel, void* y, int rows, int d, int n_exp, int top, int ff, float limit, int ff_s,
-                     float limit_s, float alpha, int mode, dli_stream_t stream);
+                     float limit_s, float alpha, int mode, int w_in, const float* sg, dli_stream_t stream);
 
 /* Pre-norm layers with a weight vector per norm.  dli_layer_close, one pass over the rows between two projections:
  *   v = x + ls * (y + bias + idw[row] * h_in)     (y == NULL: v = x; bias, idw / h_in, ls optional, fp32)
@@ -653,6 +658,16 @@ int dli_streams_close(const void* y, float* x, size_t xs_stride, int n_streams, 
                       const float* w_router, const float* logit_bias, const float* correction, float* r_wts, float* r_idw,
                       int32_t* r_sel_idx, float* r_sel_w, int n_out, int n_real, int top, int groups, int keep, float wscale,
                       int renorm, dli_stream_t stream);
+
+/* Layers whose norms are dynamic tanh maps D(z) = tanh(alpha z) * w + b (w, b [d] fp32).  One pass over the rows between two
+ * projections: with y (element type) x += mult * D_post(y); with add (fp32 rows) x += add; with next_w h = D_next(x) ->
+ * out_f (fp32) / out_e (element type), either may be NULL; with w_router the router of a mixture of experts runs on h
+ * (arguments as in dli_moe_route). */
+int dli_dyn_tanh_close(const void* y, const float* post_w, const float* post_b, float post_alpha, float mult, const float* add,
+                       float* x, const float* next_w, const float* next_b, float next_alpha, float* out_f, void* out_e, int rows,
+                       int d, int dt, const float* w_router, const float* logit_bias, const float* correction, float* r_wts,
+                       float* r_idw, int32_t* r_sel_idx, float* r_sel_w, int n_out, int n_real, int top, int groups, int keep,
+                       float wscale, int renorm, int score, const float* sg_w, float* sg, dli_stream_t stream);
 
 /* Linear attention with a decaying matrix state: S_t = diag(w_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head, S
  * [slots, H, D, V] fp32 read and advanced (an entry at position 0 starts from zero), o [rows, H*V] fp32.  q, k [H, D] and
