@@ -33,6 +33,7 @@ extra.hf_gpu : transformers' own generate (bf16, sdpa) on the same GPU and shape
 from __future__ import annotations
 
 import argparse
+import dataclasses
 import json
 import os
 import statistics
@@ -603,7 +604,7 @@ def run_togalorn_compare(args, peaks):
     return out
 
 
-def togalorn_kernel_times(eng, spec, T, peaks):
+def togalorn_kernel_times(eng, spec, T, peaks, timer=None):
     """Each kernel of the Togalorn mechanisms alone at the step sizes of the comparison: a T-token portion (prefill) and
     one token after T (decode), against its algorithmic HBM bytes or FLOPs and the measured peaks."""
     from dli_b200 import ops
@@ -614,7 +615,7 @@ def togalorn_kernel_times(eng, spec, T, peaks):
     hbm, tc = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
     res = {}
 
-    def timeit(fn, n=5, reps=10):
+    def eager(fn, n=5, reps=10):
         fn()
         return statistics.median(ev_time_ms(lambda: [fn() for _ in range(reps)]) for _ in range(n)) / reps
 
@@ -633,6 +634,7 @@ def togalorn_kernel_times(eng, spec, T, peaks):
     eng.kv.commit()
     eb = 2
     for tag, rows, start in (("prefill", T, 0), ("decode", 1, T)):
+        timeit = timer or eager
         eng._workspace(rows)
         row_ent = torch.zeros(rows, dtype=torch.int32, device=dev)
         ent = torch.tensor([slot, 0, rows, start], dtype=torch.int32, device=dev)
@@ -953,7 +955,7 @@ def run_gimudra_compare(args, peaks):
     return out
 
 
-def gimudra_kernel_times(eng, spec, T, peaks):
+def gimudra_kernel_times(eng, spec, T, peaks, timer=None):
     """Each kernel of the Gimudra mechanisms alone at the step sizes of the comparison: a T-token portion (prefill) and
     the prompt's last token alone (decode), against its algorithmic HBM bytes or FLOPs and the measured peaks."""
     from dli_b200 import ops
@@ -965,7 +967,7 @@ def gimudra_kernel_times(eng, spec, T, peaks):
     hbm, tc = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
     res = {}
 
-    def timeit(fn, n=5, reps=10):
+    def eager(fn, n=5, reps=10):
         fn()
         return statistics.median(ev_time_ms(lambda: [fn() for _ in range(reps)]) for _ in range(n)) / reps
 
@@ -982,6 +984,7 @@ def gimudra_kernel_times(eng, spec, T, peaks):
     eng.kv.commit()
     eb = 2
     for tag, rows, start in (("prefill", T, 0), ("decode", 1, T - 1)):  # the decode row sees a whole block of keys
+        timeit = timer or eager
         eng._workspace(rows)
         row_ent = torch.zeros(rows, dtype=torch.int32, device=dev)
         ent = torch.tensor([slot, 0, rows, start], dtype=torch.int32, device=dev)
@@ -1265,6 +1268,182 @@ def salizen_kernel_times(eng, spec, T, peaks):
     return res
 
 
+# ---------------------------------------------------------------------------------- Finezen beside Togalorn and Gimudra
+def finezen_config(width, heads, kv, hd, ff, layers, vocab, window=512):
+    """The Finezen design at the sizes of a Llama layer: windowed attention with the Llama layer's heads (half of a head rotated)
+    and latent attention with as many heads of the same size, a 512-wide latent and a window twice as wide, both with the Togalorn
+    comparison's mixture (8 experts of size ff/4, 2 per token, beside a shared expert of size ff/2); the two layers run layers/2
+    times."""
+    mlp = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 8, "top": 2}, "shared": {"ff": ff // 2}}
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"heads": heads, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": window},
+                     "rot": {"base": 500000.0, "dims": hd // 2, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
+    lat = {"type": "latent_attention", "mlp": mlp,
+           "mixer": {"heads": heads, "dim": hd, "vdim": hd, "kv_rank": 512, "q_rank": width // 2, "scale": hd ** -0.5, "mask": {"size": 2 * window}}}
+    return {"architecture": "Finezen", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "residual_mult": 0.7, "loop": {"start": 0, "stop": 2, "times": layers // 2}, "layers": [att, lat]}
+
+
+def graph_timer(fn, n=5, reps=20):
+    """ms per call with the calls replayed as one CUDA graph, so that short kernels are not timed as their launches
+    (operands stay in L2 where they fit; the weights of the mixtures do not)."""
+    fn()
+    torch.cuda.synchronize()
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g):
+        for _ in range(reps):
+            fn()
+    g.replay()
+    ms = statistics.median(ev_time_ms(g.replay) for _ in range(n)) / reps
+    del g
+    return ms
+
+
+def run_finezen_compare(args, peaks):
+    """Prefill and decode throughput of the Finezen design beside the framework's closest models on RaggedEngine — the
+    Togalorn design (latent attention, a mixture beside a shared expert, looped layers) and the Gimudra design (masked attention,
+    pre-normed layers closed by one kernel) — at equal layer sizes and depth, random weights, plus each kernel of the new
+    mechanisms alone against its roofline.  One JSON line; the default workload of this file is untouched."""
+    from dli_b200 import finezen, gimudra, togalorn
+    from dli_b200.ragged_engine import RaggedEngine
+
+    T, K, W = args.ctx, args.steps, args.warmup
+    out = {"metric": "finezen_vs_togalorn_gimudra", "unit": "tokens/s", "ctx": T, "steps": K, "warmup": W, "dtype": "bf16",
+           "data": "synthetic", "peaks": peaks, "sizes": {}}
+    names = args.hybrid_sizes.split(",")
+    if len(names) > 1:
+        import subprocess
+        for name in names:
+            cmd = [sys.executable, os.path.abspath(__file__), "--compare-finezen", "--hybrid-sizes", name, "--steps", str(K),
+                   "--warmup", str(W), "--ctx", str(T), "--batch", str(args.batch), "--page-size", str(args.page_size)]
+            p = subprocess.run(cmd, capture_output=True, text=True, check=True)
+            out["sizes"].update(json.loads(p.stdout.strip().splitlines()[-1])["sizes"])
+        return out
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    for name in names:
+        width, heads, kv, hd, ff, layers, vocab = HYBRID_SIZES[name]
+        mods = ((finezen, finezen_config(width, heads, kv, hd, ff, layers, vocab), "finezen"),
+                (togalorn, togalorn_config(width, heads, kv, hd, ff, layers, vocab), "togalorn"),
+                (gimudra, gimudra_config(width, heads, kv, hd, ff, layers, vocab), "gimudra"))
+        res = {}
+        for mod, cfg, tag in mods:
+            spec = mod.spec_from_config(cfg)
+            eng = RaggedEngine(spec, max_batch=max(args.batch, 8), max_seq_len=T + K + W + 64, page_size=args.page_size)
+            eng.load_tensors(mod.model_tensors(spec, mod.random_state_dict(spec, seed=1, std=0.02, device="cuda")))
+            res.update(ragged_throughput(eng, vocab, T, K, W, args.batch, tag, flush))
+            res[f"{tag}_kernels"] = {"finezen": finezen_kernel_times, "togalorn": togalorn_kernel_times,
+                                     "gimudra": gimudra_kernel_times}[tag](eng, spec, T, peaks, timer=graph_timer)
+            eng.unload()
+            del eng
+            torch.cuda.empty_cache()
+        out["sizes"][name] = res
+    return out
+
+
+def finezen_kernel_times(eng, spec, T, peaks, timer=graph_timer):
+    """Each kernel of the Finezen mechanisms alone at the step sizes of the comparison: a T-token portion (prefill) and
+    the prompt's last token alone (decode), against its algorithmic HBM bytes or FLOPs and the measured peaks."""
+    from dli_b200 import ops
+
+    dev, E, W = eng.device, eng.dtype, spec.width
+    hbm, tc = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    res = {}
+
+    def put(key, ms, byt=None, flops=None):
+        d = {"ms": round(ms, 4)}
+        if byt is not None:
+            d["of_hbm"] = round(byt / (ms / 1e3) / hbm, 3)
+        if flops is not None:
+            d["of_bf16_peak"] = round(flops / (ms / 1e3) / tc, 4)
+        res[key] = d
+
+    li_a = next(i for i, L in enumerate(spec.layers) if L.mixer.kind == "attention")
+    li_l = next(i for i, L in enumerate(spec.layers) if L.mixer.kind == "latent_attention")
+    slot = eng.open_sequence()
+    eng.kv.reserve(slot, T + 1)
+    eng.kv.commit()
+    eb = 2
+    for tag, rows, start in (("prefill", T, 0), ("decode", 1, T - 1)):
+        timeit = timer
+        eng._workspace(rows)
+        row_ent = torch.zeros(rows, dtype=torch.int32, device=dev)
+        ent = torch.tensor([slot, 0, rows, start], dtype=torch.int32, device=dev)
+        d_tiles = torch.tensor([[0, q0] for q0 in range(0, rows, 64)] if rows > 1 else [], dtype=torch.int32, device=dev).flatten()
+        views = (None, row_ent, ent, None, d_tiles)
+        eng._step_pages = (min(eng.kv.owned[slot]), max(eng.kv.owned[slot]))
+        eng._step_spans = [(slot, start, start + rows)]
+        x, add = torch.randn(rows, W, device=dev), torch.randn(rows, W, device=dev)
+        he = torch.empty(rows, W, dtype=E, device=dev)
+        y = torch.randn(rows, W, device=dev).to(E)
+        P, e = eng.layers[li_a], spec.layers[li_a].moe
+        close = dict(y=y, post=P["norm1b"], mult=0.01, nxt=P["norm2"], out_e=he)
+        vec = 16 * W                                                    # both maps' weights and offsets
+        put(f"{tag}_close_norm", timeit(lambda: ops.dyn_tanh_close(x, **close)), byt=rows * W * (8 + 2 * eb) + vec)
+        put(f"{tag}_close_add_norm", timeit(lambda: ops.dyn_tanh_close(x, add=add, **close)), byt=rows * W * (12 + 2 * eb) + vec)
+        route = eng._route_args(e, P, rows)
+        put(f"{tag}_close_norm_route", timeit(lambda: ops.dyn_tanh_close(x, route=route, **close)),
+            byt=rows * W * (8 + 2 * eb) + vec + P["w_router"].numel() * 4)
+        # windowed attention: norms over the whole projections, rotation, append; scores with a sink; a gate per head
+        m, PP = spec.layers[li_a].mixer, P
+        proj = (0.5 * torch.randn(rows, P["w_proj"].shape[0], device=dev)).to(E)
+        mix = torch.empty(rows, m.heads * m.vdim, dtype=E, device=dev)
+        qbuf = torch.empty(rows, m.heads * m.dim, device=dev)
+        kc, vc = eng.kv.k[eng.kv_index[li_a]], eng.kv.v[eng.kv_index[li_a]]
+        cos_t, sin_t = eng._table(m.rot_base, m.rot_dims, m.rot_scaling)
+        off, win = PP["off"], m.window or T
+        for whole in (True, False):
+            qn, kn = (PP["q_norm"], PP["k_norm"]) if whole else (PP["q_norm"][:m.dim].contiguous(), PP["k_norm"][:m.dim].contiguous())
+            put(f"{tag}_attn_prep" + ("" if whole else "_norm_per_head"),
+                timeit(lambda: ops.attn_prep_append(proj, qbuf, kc, vc, row_ent, ent, eng.kv.page_table, m.heads, m.kv_heads, m.dim, m.vdim,
+                                                    m.rot_dims, off["q"], off["k"], off["v"], qn, kn, 1e-6, cos_t, sin_t, None, None,
+                                                    halves=True, whole_norm=whole)),
+                byt=rows * (m.heads * m.dim * (eb + 4) + m.kv_heads * (m.dim + m.vdim) * 2 * eb))
+        pairs = sum(min(t + 1, win) for t in range(start, start + rows))
+        kw = dict(window=m.window, sink=PP["sink"], g_off=off["g"])
+        if rows > 1:
+            ms = timeit(lambda: ops.attn_ragged_tc(qbuf, kc, vc, proj, mix, ent, d_tiles, eng.kv.page_table, m.heads, m.kv_heads, m.dim, m.vdim,
+                                                   m.scale, **kw))
+            put(f"{tag}_attn", ms, flops=2 * pairs * m.heads * (m.dim + m.vdim))
+        else:
+            splits = max(1, min(16, (4 * eng._sms) // (rows * m.heads), (win + 31) // 32))
+            ms = timeit(lambda: ops.attn_ragged(qbuf, kc, vc, proj, mix, row_ent, ent, eng.kv.page_table, m.heads, m.kv_heads, m.dim, m.vdim,
+                                                m.scale, splits=splits, part=eng._apart_att if splits > 1 else None, **kw))
+            put(f"{tag}_attn", ms, byt=min(start + 1, win) * m.kv_heads * (m.dim + m.vdim) * eb)
+        # latent attention: everything between the input projection and the output projection, with the window and without
+        PL = eng.layers[li_l]
+        proj = (0.5 * torch.randn(rows, PL["w_proj"].shape[0], device=dev)).to(E)
+        m0 = spec.layers[li_l].mixer
+        mix = torch.empty(rows, m0.heads * m0.vdim, dtype=E, device=dev)
+        for m, key in ((m0, f"{tag}_latent_attention_all"), (dataclasses.replace(m0, window=0), f"{tag}_latent_attention_all_no_window")):
+            win = m.window or T
+            ms = timeit(lambda: eng._latent_attention(li_l, m, PL, proj, mix, rows, views, rows > 1), n=3, reps=3)
+            if rows > 1:
+                pairs = sum(min(t + 1, win) for t in range(rows))
+                put(key, ms, flops=2 * pairs * m.heads * (m.dim + m.vdim) + 2 * rows * (m.q_rank * m.heads * m.dim + m.kv_rank * m.heads * (m.dim + m.vdim)))
+            else:
+                put(key, ms, byt=min(start + 1, win) * m.kv_rank * eb + (PL["w_uq"].numel() + PL["uk"].numel() + PL["uv"].numel()) * eb)
+        # the experts
+        gu = torch.empty(rows, P["w_gu"].shape[0], dtype=E, device=dev)
+        act = torch.empty(rows, e.total_ff, dtype=E, device=dev)
+        y2 = torch.empty(rows, W, dtype=E, device=dev)
+        more = dict(silu=True, weight_in=True, sg=route["sg"])
+        ms_gu = timeit(lambda: eng._lin(he, P["w_gu"], gu), n=3, reps=3)
+        ms_act = timeit(lambda: ops.moe_act(gu, route["wts"], act, e.experts, e.ff, 0.0, e.shared_ff, **more))
+        ms_dn = timeit(lambda: eng._lin(act, P["w_down"], y2), n=3, reps=3)
+        put(f"{tag}_moe_act", ms_act, byt=rows * (e.total_ff + 2 * (e.top * e.ff + e.shared_ff)) * eb)
+        if rows > 1:
+            put(f"{tag}_moe_projections", ms_gu + ms_dn, flops=2 * rows * 3 * W * (e.top * e.ff + e.shared_ff))
+            res[f"{tag}_moe_projections"]["of_bf16_peak_all_experts"] = round(2 * rows * 3 * W * e.total_ff / ((ms_gu + ms_dn) / 1e3) / tc, 4)
+        else:
+            put(f"{tag}_moe_projections_all_experts", ms_gu + ms_dn, byt=3 * W * e.total_ff * eb)
+            act_sel = torch.empty(rows, e.top * e.ff + e.shared_ff, dtype=E, device=dev)
+            ms = timeit(lambda: ops.moe_sel(he, P["w_gu"], P["w_down"], route["sel_idx"], route["sel_w"], act_sel, y2, e.experts, e.top,
+                                            e.ff, 0.0, e.shared_ff, **more))
+            put(f"{tag}_moe_chosen_experts", ms, byt=3 * W * (e.top * e.ff + e.shared_ff) * eb)
+    eng.close_sequence(slot)
+    return res
+
+
 def hybrid_kernel_times(eng, spec, T, peaks):
     """Each kernel of the ragged path alone at the step sizes of the comparison: a T-token portion (prefill) and one
     token after T (decode), against its algorithmic HBM bytes (or FLOPs) and the measured peaks."""
@@ -1408,6 +1587,8 @@ def main():
                     help="prefill / decode throughput of the Gimudra design beside the Togalorn and Sokevik designs at equal sizes")
     ap.add_argument("--compare-salizen", action="store_true",
                     help="prefill / decode throughput of the Salizen design beside the Togalorn and Gimudra designs at equal sizes")
+    ap.add_argument("--compare-finezen", action="store_true",
+                    help="prefill / decode throughput of the Finezen design beside the Togalorn and Gimudra designs at equal sizes")
     ap.add_argument("--hybrid-sizes", default="1b,8b")
     args = ap.parse_args()
 
@@ -1442,6 +1623,10 @@ def main():
     if args.compare_salizen:
         if rank == 0:
             print(json.dumps(run_salizen_compare(args, peaks)), flush=True)
+        return
+    if args.compare_finezen:
+        if rank == 0:
+            print(json.dumps(run_finezen_compare(args, peaks)), flush=True)
         return
     if world > 1 or args.gpus > 1:
         from dli_b200.pipeline import run_pipeline_bench
