@@ -396,7 +396,7 @@ attn_ragged_kernel(const float* __restrict__ qbuf, const E* __restrict__ kc, con
 }
 
 // Adds the partial sums of a row's key splits: o = sum_z e^(m_z - M) o_z / sum_z e^(m_z - M) l_z, then the same
-// epilogue (turn back, gate).  One CTA per (row, head).
+// epilogue (turn back, gate).  CTAs per (row, head, 256 value dimensions).
 template <typename E>
 __global__ void __launch_bounds__(kAttnThreads)
 attn_ragged_merge_kernel(const E* __restrict__ proj, E* __restrict__ out, AttnRun a) {
@@ -422,17 +422,18 @@ attn_ragged_merge_kernel(const E* __restrict__ proj, E* __restrict__ out, AttnRu
   const int pos = e.w + (row - e.y);
   const float inv = 1.f / L;
   E* orow = out + (size_t)row * a.ldo + h * a.V;
-  for (int i = tid; i < a.V / 2; i += kAttnThreads) {
+  for (int i = blockIdx.z * kAttnThreads + tid; i < a.V / 2; i += kAttnThreads * gridDim.z) {
     float u = 0.f, v = 0.f;
-    for (int z0 = 0; z0 < a.splits; z0 += 8) {  // eight splits' loads in flight together
-      float2 f[8];
+    constexpr int ZR = 16;
+    for (int z0 = 0; z0 < a.splits; z0 += ZR) {  // sixteen splits' loads in flight together
+      float2 f[ZR];
 #pragma unroll
-      for (int k = 0; k < 8; ++k) {
+      for (int k = 0; k < ZR; ++k) {
         const int z = min(z0 + k, a.splits - 1);
         f[k] = *reinterpret_cast<const float2*>(pr + (size_t)z * (a.V + 2) + 2 * i);
       }
 #pragma unroll
-      for (int k = 0; k < 8; ++k)
+      for (int k = 0; k < ZR; ++k)
         if (z0 + k < a.splits) { u = fmaf(wz[z0 + k], f[k].x, u); v = fmaf(wz[z0 + k], f[k].y, v); }
     }
     u *= inv; v *= inv;
@@ -493,26 +494,30 @@ attn_shared_kv_kernel(const float* __restrict__ qbuf, const E* __restrict__ kc, 
   }
   __syncthreads();
   for (int j0 = jb; j0 <= je; j0 += kAttnThreads) {
-    const int j = j0 + tid;
-    const bool valid = j <= je;
+    // a pass of at most 64 / 32 keys (the key splits of decode rows): 2 / 4 neighbouring threads share a key's dot products,
+    // each taking every second / fourth 16-byte piece of the row
+    const int n_keys = min(kAttnThreads, je - j0 + 1);
+    const int tpk = n_keys <= 32 ? 4 : (n_keys <= 64 ? 2 : 1);
+    const int kidx = tid / tpk, part = tid - kidx * tpk, step = 8 * tpk;
+    const int j = j0 + kidx;
     float s[HPC];
 #pragma unroll
     for (int h = 0; h < HPC; ++h) s[h] = 0.f;
-    if (valid) {
+    if (j <= je) {
       const E* kr = kc + ((size_t)pt[j / a.page_size] * a.page_size + j % a.page_size) * a.D;
-      int c = 0;
-      for (; c + 32 <= a.D; c += 32) {  // four 16-byte key loads in flight before the first is used
+      int c = part * 8;
+      for (; c + 3 * step < a.D; c += 4 * step) {  // four 16-byte key loads in flight before the first is used
         float f[4][8];
 #pragma unroll
-        for (int u = 0; u < 4; ++u) load8(kr + c + 8 * u, f[u]);
+        for (int u = 0; u < 4; ++u) load8(kr + c + step * u, f[u]);
 #pragma unroll
         for (int u = 0; u < 4; ++u)
 #pragma unroll
           for (int h = 0; h < HPC; ++h)
 #pragma unroll
-            for (int i = 0; i < 8; ++i) s[h] = fmaf(q[h * a.D + c + 8 * u + i], f[u][i], s[h]);
+            for (int i = 0; i < 8; ++i) s[h] = fmaf(q[h * a.D + c + step * u + i], f[u][i], s[h]);
       }
-      for (; c < a.D; c += 8) {
+      for (; c < a.D; c += step) {
         float f[8];
         load8(kr + c, f);
 #pragma unroll
@@ -521,6 +526,14 @@ attn_shared_kv_kernel(const float* __restrict__ qbuf, const E* __restrict__ kc, 
           for (int i = 0; i < 8; ++i) s[h] = fmaf(q[h * a.D + c + i], f[i], s[h]);
       }
     }
+    if (tpk > 1) {
+#pragma unroll
+      for (int h = 0; h < HPC; ++h) {
+        s[h] += __shfl_xor_sync(0xffffffffu, s[h], 1);
+        if (tpk > 2) s[h] += __shfl_xor_sync(0xffffffffu, s[h], 2);
+      }
+    }
+    const bool valid = j <= je && part == 0;
 #pragma unroll
     for (int h = 0; h < HPC; ++h) {
       if (!valid) s[h] = -INFINITY;
@@ -535,7 +548,7 @@ attn_shared_kv_kernel(const float* __restrict__ qbuf, const E* __restrict__ kc, 
       const float m_new = fmaxf(m[h], mx);
       corr[h] = (m[h] == -INFINITY) ? 0.f : expf(m[h] - m_new);
       const float w = valid ? expf(s[h] - m_new) : 0.f;
-      p[h * kAttnThreads + tid] = w;
+      if (part == 0) p[h * kAttnThreads + kidx] = w;
       const float ws = warp_sum(w);
       if (lane == 0) red[HPC * 4 + h * 4 + warp] = ws;
       m[h] = m_new;
@@ -948,8 +961,9 @@ int dli_attn_ragged(const float* qbuf, const void* k_cache, const void* v_cache,
   if (dt == 0) DLI_LAUNCH("attn_ragged", attn_ragged_kernel<bf16>, dim3(rows, H, splits), dim3(kAttnThreads), smem, s, qbuf, (const bf16*)k_cache, (const bf16*)v_cache, (const bf16*)proj, (bf16*)out, a);
   else DLI_LAUNCH("attn_ragged", attn_ragged_kernel<float>, dim3(rows, H, splits), dim3(kAttnThreads), smem, s, qbuf, (const float*)k_cache, (const float*)v_cache, (const float*)proj, (float*)out, a);
   if (splits > 1) {
-    if (dt == 0) DLI_LAUNCH("attn_ragged_merge", attn_ragged_merge_kernel<bf16>, dim3(rows, H), dim3(kAttnThreads), 0, s, (const bf16*)proj, (bf16*)out, a);
-    else DLI_LAUNCH("attn_ragged_merge", attn_ragged_merge_kernel<float>, dim3(rows, H), dim3(kAttnThreads), 0, s, (const float*)proj, (float*)out, a);
+    const int mz = (V / 2 + kAttnThreads - 1) / kAttnThreads;
+    if (dt == 0) DLI_LAUNCH("attn_ragged_merge", attn_ragged_merge_kernel<bf16>, dim3(rows, H, mz), dim3(kAttnThreads), 0, s, (const bf16*)proj, (bf16*)out, a);
+    else DLI_LAUNCH("attn_ragged_merge", attn_ragged_merge_kernel<float>, dim3(rows, H, mz), dim3(kAttnThreads), 0, s, (const float*)proj, (float*)out, a);
   }
   return DLI_OK;
 }
